@@ -394,19 +394,22 @@ __global__ void __launch_bounds__(256) add_bias_kernel(float* __restrict__ x, co
 // by the angle position * inv_freq[i]; queries to q_out [T, H * D], keys and values to their page. Everything is float
 // until the one rounding at the store. The row (with its bias) and the token's cosines and sines are kept in shared
 // memory, so the sums are read from memory once (rows of up to 200 KB). With head_norm every query and key head is
-// instead divided, after its rotation, by its own root mean square over its dim true elements, without a weight.
+// instead divided, after its rotation, by its own root mean square over its dim true elements, without a weight; with
+// head_norm 2 before its rotation, and multiplied by a weight [D] that all query (all key) heads share. With keys_are_values
+// the row ends with the keys, [T, (H + G) * D], and the value pages take the keys as projected, before norm and rotation.
 template <typename T>
 __global__ void __launch_bounds__(512) qk_prepare_kernel(
     const float* __restrict__ sums, int stride, const float* __restrict__ bias, const int* __restrict__ positions,
     const int* __restrict__ token_row, int H, int G, int D, int dim, const float* __restrict__ q_weight, const float* __restrict__ k_weight,
     float eps, const float* __restrict__ inv_freq, int rot, T* __restrict__ q_out, int q_stride, T* __restrict__ kc, T* __restrict__ vc,
-    const int* __restrict__ block_table, int bt_width, int ps, int num_pages, int* __restrict__ errors, int head_norm) {
+    const int* __restrict__ block_table, int bt_width, int ps, int num_pages, int* __restrict__ errors, int head_norm, int keys_are_values) {
   __shared__ float red[32];
   extern __shared__ float dyn[];            // [half] cosines, [half] sines of this token's angles, then the token's row with its bias
   const int t = blockIdx.x;
   const float* row = sums + (size_t)t * stride;
   const int nq = H * D, nk = G * D, half = rot >> 1;
-  const int n_all = nq + 2 * nk;
+  const int n_all = nq + (keys_are_values ? 1 : 2) * nk;
+  const bool whole_norm = head_norm == 0;
   float* cs_table = dyn;
   float* vals = dyn + (rot > 0 ? rot : 2);
   const int pos = positions[t];
@@ -421,8 +424,8 @@ __global__ void __launch_bounds__(512) qk_prepare_kernel(
     else if (i < nq + nk) sk += v * v;
   }
   float inv_q = 1.f, inv_k = 1.f;
-  if (q_weight != nullptr) inv_q = 1.0f / sqrtf(block_sum(sq, red) / (float)(H * dim) + eps);
-  if (k_weight != nullptr && G > 0) inv_k = 1.0f / sqrtf(block_sum(sk, red) / (float)(G * dim) + eps);
+  if (q_weight != nullptr && whole_norm) inv_q = 1.0f / sqrtf(block_sum(sq, red) / (float)(H * dim) + eps);
+  if (k_weight != nullptr && whole_norm && G > 0) inv_k = 1.0f / sqrtf(block_sum(sk, red) / (float)(G * dim) + eps);
   __syncthreads();                          // the table and the row are whole
   // A warp takes a head at a time, a lane an element; an element below rot / 2 is turned together with its partner rot / 2
   // further on, so every value is normalised once. Heads 0 .. H-1 are queries, the G after them keys.
@@ -436,10 +439,14 @@ __global__ void __launch_bounds__(512) qk_prepare_kernel(
     const bool is_q = head < H;
     if (!is_q && !page_ok) continue;
     const float* w = is_q ? q_weight : k_weight;
-    const float inv = is_q ? inv_q : inv_k;
-    const int base = head * D, w_base = is_q ? base : base - nq;
+    float inv = is_q ? inv_q : inv_k;
+    const int base = head * D, w_base = head_norm == 2 ? 0 : (is_q ? base : base - nq);
     T* dst = is_q ? q_out + (size_t)t * q_stride + base : kc + (((size_t)page * G + (head - H)) * ps + within) * D;
-    if (head_norm) {
+    if (head_norm == 2) {
+      float ss = 0.f;
+      for (int d = lane; d < D; d += 32) ss += vals[base + d] * vals[base + d];      // (zero beyond the head's true size)
+      inv = 1.0f / sqrtf(warp_sum(ss) / (float)dim + eps);
+    } else if (head_norm) {
       // the head is turned in place in shared memory (a lane turns an element together with its partner), its squares are
       // summed over the warp, and the quotient is stored
       float ss = 0.f;
@@ -478,9 +485,10 @@ __global__ void __launch_bounds__(512) qk_prepare_kernel(
     }
   }
   if (!page_ok) return;
+  const float* values = vals + nq + (keys_are_values ? 0 : nk);
   for (int i = threadIdx.x; i < nk; i += blockDim.x) {
     const int g = i / D, d = i - g * D;
-    vc[(((size_t)page * G + g) * ps + within) * D + d] = from_float<T>(vals[nq + nk + i]);
+    vc[(((size_t)page * G + g) * ps + within) * D + d] = from_float<T>(values[i]);
   }
 }
 
@@ -542,19 +550,21 @@ SB_EXPORT int sb_add_bias(float* x, const float* bias, int n_rows, int cols, cud
   return 0;
 }
 
-// bias float [(H + 2 G) * D] or null; q_weight float [H * D], k_weight float [G * D] or null (no norm of that side);
-// inv_freq float [>= rot / 2]; G = 0 writes no cache.
+// bias float [(H + 2 G) * D] or null; q_weight float [H * D], k_weight float [G * D] or null (no norm of that side); with
+// head_norm 2 both are float [D], and with keys_are_values rows and bias have (H + G) * D columns; inv_freq float [>= rot / 2];
+// G = 0 writes no cache.
 SB_EXPORT int sb_qk_prepare(const float* sums, int stride, const float* bias, const int* positions, const int* token_row, int H, int G, int D,
                             int dim, const float* q_weight, const float* k_weight, float eps, const float* inv_freq, int rot, void* q_out,
                             int q_stride, void* kc, void* vc, const int* block_table, int bt_width, int ps, int num_pages, int* errors,
-                            int n_tokens, int dtype, int head_norm, cudaStream_t stream) {
+                            int n_tokens, int dtype, int head_norm, int keys_are_values, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
-  if (H <= 0 || G < 0 || D <= 0 || dim <= 0 || dim > D || stride < (H + 2 * G) * D || q_stride < H * D) return SB_ERR_SHAPE;
+  const int n_all = (H + (keys_are_values ? 1 : 2) * G) * D;
+  if (H <= 0 || G < 0 || D <= 0 || dim <= 0 || dim > D || stride < n_all || head_norm < 0 || head_norm > 2 || (head_norm == 2 && (!q_weight || (G > 0 && !k_weight))) || q_stride < H * D) return SB_ERR_SHAPE;
   if (rot < 0 || (rot & 1) || rot > dim || (rot > 0 && !inv_freq)) return SB_ERR_SHAPE;
   if (G > 0 && (ps <= 0 || bt_width <= 0 || !kc || !vc || !errors)) return SB_ERR_SHAPE;
-  const size_t smem = ((size_t)(rot > 0 ? rot : 2) + (size_t)(H + 2 * G) * D) * sizeof(float);
+  const size_t smem = ((size_t)(rot > 0 ? rot : 2) + (size_t)n_all) * sizeof(float);
   if (smem > 200 * 1024) return SB_ERR_LIMIT;
-  const int threads = (H + 2 * G) * D >= 2048 ? 512 : 256;
+  const int threads = n_all >= 2048 ? 512 : 256;
   if (smem > 48 * 1024) {
     cudaFuncSetAttribute(qk_prepare_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     cudaFuncSetAttribute(qk_prepare_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -562,11 +572,11 @@ SB_EXPORT int sb_qk_prepare(const float* sums, int stride, const float* bias, co
   if (dtype == SB_DTYPE_F32)
     qk_prepare_kernel<float><<<n_tokens, threads, smem, stream>>>(sums, stride, bias, positions, token_row, H, G, D, dim, q_weight, k_weight, eps,
                                                             inv_freq, rot, (float*)q_out, q_stride, (float*)kc, (float*)vc, block_table,
-                                                            bt_width, ps, num_pages, errors, head_norm);
+                                                            bt_width, ps, num_pages, errors, head_norm, keys_are_values);
   else if (dtype == SB_DTYPE_BF16)
     qk_prepare_kernel<__nv_bfloat16><<<n_tokens, threads, smem, stream>>>(sums, stride, bias, positions, token_row, H, G, D, dim, q_weight, k_weight,
                                                                     eps, inv_freq, rot, (__nv_bfloat16*)q_out, q_stride, (__nv_bfloat16*)kc,
-                                                                    (__nv_bfloat16*)vc, block_table, bt_width, ps, num_pages, errors, head_norm);
+                                                                    (__nv_bfloat16*)vc, block_table, bt_width, ps, num_pages, errors, head_norm, keys_are_values);
   else
     return SB_ERR_DTYPE;
   SB_LAUNCH_CHECK();

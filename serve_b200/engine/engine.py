@@ -62,13 +62,14 @@ class Engine:
         # the libraries the model's parts will call are compiled side by side now, not one after the other at first use
         prepare = getattr(kernels, "prepare", None)
         if prepare is not None:
-            dims, libs = set(), set()
+            dims, libs, talk = set(), set(), set()
             for part in self.model.all_parts():
                 needs = part.kernel_needs()
                 dims.update(needs.get("attention_head_dims", ()))
                 libs.update(needs.get("libraries", ()))
-            if dims or libs:
-                prepare(sorted(dims), sorted(libs))
+                talk.update(needs.get("talking_head_dims", ()))
+            if dims or libs or talk:
+                prepare(sorted(dims), sorted(libs), sorted(talk))
         self.cache: Optional[CacheManager] = None
         self.stepper: Optional[Stepper] = None
         self.max_context = min(self.engine_config.max_context or self.spec.max_position, self.spec.max_position)

@@ -82,13 +82,18 @@ def experts_job():
 
 
 def projection_job():
-    """Layer norm, whole-projection query/key norm with temperature, latent-attention preparation, gated activations."""
-    return {"name": "sb_prep", "sources": ["projection_ops.cu"]}
+    """Layer norm, grouped norm, whole-projection query/key norm with temperature, latent-attention preparation, activations."""
+    return {"name": "sb_prep", "sources": ["projection_ops.cu", "grouped_norm.cu"]}
 
 
 def attention_job(head_dim: int):
     return {"name": f"sb_attention_hd{head_dim}", "sources": ["attention_simt.cu", "attention_mma.cu", "attention_tc.cu"],
             "defines": [f"SB_HEAD_DIM={head_dim}"]}
+
+
+def talking_attention_job(head_dim: int):
+    """Attention whose heads' weights are mixed before the values (built when a model first asks for it)."""
+    return {"name": f"sb_talk_hd{head_dim}", "sources": ["talking_attention.cu"], "defines": [f"SB_HEAD_DIM={head_dim}"]}
 
 
 def layer_run_job(head_dim: int):
@@ -124,6 +129,7 @@ class LayerRunPlan:
 def all_jobs():
     """Every library the engine can ask for (the build check compiles them all)."""
     return (core_jobs() + [sequence_job(), experts_job(), projection_job()] + [attention_job(d) for d in SUPPORTED_HEAD_DIMS]
+            + [talking_attention_job(d) for d in SUPPORTED_HEAD_DIMS]
             + [layer_run_job(d) for d in LAYER_RUN_HEAD_DIMS])
 
 
@@ -170,6 +176,7 @@ class CudaKernels:
         self._seq = None                     # the library of sequence_job(), loaded at first use
         self._moe = None                     # the library of experts_job(), loaded at first use
         self._prep = None                    # the library of projection_job(), loaded at first use
+        self._talk: Dict[int, ctypes.CDLL] = {}     # libraries of talking_attention_job(), by head size
         self._stack: Dict[int, ctypes.CDLL] = {}
         self._stack_sync = None              # two counters of the layer-run kernel's grid barrier (zero between launches)
         self._stack_partials = None
@@ -208,13 +215,26 @@ class CudaKernels:
             lib.sb_attention_mma_scratch_bytes.restype = ctypes.c_longlong
         return lib
 
-    def prepare(self, head_dims=(), libraries=()) -> None:
-        """Build side by side, and load, what a model is going to call: attention libraries for ``head_dims`` and the
-        optional libraries named ("seq", "moe", "prep"). Without this each is built when first called."""
+    def _talk_lib(self, head_dim: int):
+        lib = self._talk.get(head_dim)
+        if lib is None:
+            self.check_attention_shape(1, 1, head_dim)
+            job = talking_attention_job(head_dim)
+            job["verbose"] = self._verbose
+            path = build.build_library(**job)
+            self.paths[job["name"]] = path
+            lib = self._talk[head_dim] = ctypes.CDLL(path)
+        return lib
+
+    def prepare(self, head_dims=(), libraries=(), talking_head_dims=()) -> None:
+        """Build side by side, and load, what a model is going to call: attention libraries for ``head_dims``, those with mixed
+        heads for ``talking_head_dims`` and the optional libraries named ("seq", "moe", "prep"). Without this each is built when
+        first called."""
         named = {"seq": sequence_job, "moe": experts_job, "prep": projection_job}
         jobs = [attention_job(d) for d in sorted(set(head_dims)) if d not in self._attn]
-        for d in head_dims:
+        for d in list(head_dims) + list(talking_head_dims):
             self.check_attention_shape(1, 1, d)
+        jobs += [talking_attention_job(d) for d in sorted(set(talking_head_dims)) if d not in self._talk]
         jobs += [named[n]() for n in sorted(set(libraries)) if getattr(self, "_" + n) is None]
         if not jobs:
             return
@@ -223,6 +243,8 @@ class CudaKernels:
         self.paths.update(build.build_many(jobs))
         for d in head_dims:
             self._attention_lib(d)
+        for d in talking_head_dims:
+            self._talk_lib(d)
         for n in libraries:
             getattr(self, f"_{n}_lib")()
 
@@ -342,6 +364,27 @@ class CudaKernels:
         _check(self._prep_lib().sb_add_layernorm(_p(x), _p(delta), _p(rows), _p(weight), _DT[weight.dtype], _p(out), rows.shape[0],
                                                  x.shape[1], ctypes.c_float(eps), _DT[out.dtype], self._s()), "add_layernorm_rows")
 
+    def add_grouped_rmsnorm(self, x, delta, through, rows, weight, groups: int, eps: float, out) -> None:
+        """x += d; out = every one of ``groups`` equal parts of x divided by its own root mean square, times weight (float). d is
+        ``delta`` (activations or float), or, with ``through`` (the float weight of such a norm the delta still has to pass), that
+        norm of it. With ``rows`` only those rows, and x stays as it is; with x None, out = the norm of delta."""
+        if weight.dtype != torch.float32 or (through is not None and through.dtype != torch.float32):
+            raise KernelError("add_grouped_rmsnorm: the weights are float")
+        self.launches += 1
+        n_rows = rows.shape[0] if rows is not None else out.shape[0]
+        _check(self._prep_lib().sb_add_grouped_rmsnorm(
+            _p(x), _p(delta), _DT[delta.dtype] if delta is not None else 0, _p(through), _p(rows), _p(weight), _p(out), _DT[out.dtype],
+            n_rows, out.shape[1], int(groups), ctypes.c_float(eps), self._s()), "grouped norm")
+
+    def poly_norm(self, z, coef, eps: float, out) -> None:
+        """out = a N(z) + b N(z^2) + c N(z^3) + e row by row, N dividing a row by its root mean square; coef float [a, b, c, e].
+        z and out contiguous and alike; may be the same buffer."""
+        if coef.dtype != torch.float32 or z.dtype != out.dtype or z.shape != out.shape or not z.is_contiguous() or not out.is_contiguous():
+            raise KernelError("poly_norm: z and out must be contiguous and alike, the coefficients float")
+        self.launches += 1
+        _check(self._prep_lib().sb_poly_norm(_p(z), _p(coef), ctypes.c_float(eps), _p(out), z.shape[0], z.shape[1], _DT[z.dtype], self._s()),
+               "polynomial activation")
+
     def add_dynamic_tanh(self, x, delta, through, rows, params, out) -> None:
         """x += d; out = tanh(alpha x) w + b with params = float [w | b | alpha]. d is ``delta`` (activations or float), or, with
         ``through`` (the parameters of the dynamic tanh the delta still has to pass), tanh(alpha' delta) w' + b'. With ``rows``
@@ -389,12 +432,14 @@ class CudaKernels:
         _check(self._prep_lib().sb_add_bias(_p(x), _p(bias), x.shape[0], x.shape[1], self._s()), "bias")
 
     def qk_prepare(self, sums, bias, positions, token_row, heads, kv_heads, head_dim, dim, q_weight, k_weight, eps, inv_freq, rot_dims,
-                   q_out, k_cache, v_cache, block_table, page_size, head_norm: bool = False) -> None:
+                   q_out, k_cache, v_cache, block_table, page_size, head_norm: bool = False, keys_are_values: bool = False) -> None:
         """From the float sums of a fused query | key | value projection [T, (H + 2 G) * D] (heads padded to D; G = 0: queries only):
         bias added, all queries (all keys) of a token divided by their root mean square over H * dim (G * dim) true elements and
         multiplied by float weights laid out like the padded projection (None: no norm), the first rot_dims elements of every
-        query and key head rotated (pairs i, i + rot_dims / 2), queries to q_out, keys and values to their pages. ``head_norm``:
-        instead, every query and key head is divided, after its rotation, by its own root mean square over dim elements."""
+        query and key head rotated (pairs i, i + rot_dims / 2), queries to q_out, keys and values to their pages. ``head_norm``
+        True: instead, every query and key head is divided, after its rotation, by its own root mean square over dim elements;
+        "before": before its rotation, and times a weight [D] that all query (all key) heads share. ``keys_are_values``: the row ends
+        with the keys, and the value pages take them as projected (bias added)."""
         if sums.dtype != torch.float32:
             raise KernelError("qk_prepare: the projection's sums are float")
         self.launches += 1
@@ -403,7 +448,8 @@ class CudaKernels:
             _p(sums), sums.stride(0), _p(bias), _p(positions), _p(token_row), heads, kv_heads, head_dim, dim, _p(q_weight), _p(k_weight),
             ctypes.c_float(eps), _p(inv_freq), int(rot_dims), _p(q_out), q_out.stride(0), _p(k_cache if kv_heads else None),
             _p(v_cache if kv_heads else None), _p(block_table), block_table.shape[1], page_size, pages, _p(self.errors_tensor()),
-            sums.shape[0], _DT[q_out.dtype], 1 if head_norm else 0, self._s()), "query/key preparation")
+            sums.shape[0], _DT[q_out.dtype], 2 if head_norm == "before" else (1 if head_norm else 0), 1 if keys_are_values else 0, self._s()),
+            "query/key preparation")
 
     def linear_batched(self, a, w, out) -> None:
         """out[:, b] = a[:, b] @ w[b]^T for every b: a [M, B, K] and out [M, B, N] may be views of wider buffers (unit stride
@@ -721,6 +767,52 @@ class CudaKernels:
             heads, kv_heads, page_size, k_cache.shape[0], ctypes.c_float(scale), window, _p(out), shape.rows, shape.max_q,
             which, int(shape.max_kv), num_splits, _p(scratch), _p(tickets), _p(wide_rows), n_wide, _p(slopes), chunk,
             ctypes.c_float(softcap), _p(sinks), kv_div, keep_first, self._s()), "attention")
+
+    # Scratch bytes a launch of the mixed-head attention may use; a step that needs more runs in runs of tokens.
+    TALK_SCRATCH_BYTES = int(os.environ.get("SERVE_B200_TALK_SCRATCH", str(512 << 20)))
+
+    def talking_attention(self, q, k_cache, v_cache, block_table, cu_q, kv_len, positions, heads, kv_heads, head_dim, page_size, scale,
+                          talk, out, shape, chunk: int = 0, softcap: float = 0.0, sinks=None) -> None:
+        """Attention whose heads' softmax weights are mixed before they meet the values: weight_h = sum_g talk[h, g] weight_g, head h
+        then reads the values of its own kv head. q [T, H * D]; ``talk`` of q's type: [H, H] in float32, in bfloat16 [Hp, Hp] with Hp
+        the next multiple of 16 and zeros beyond H. chunk, softcap and sinks as in ``attention``."""
+        lib = self._talk_lib(head_dim)
+        group = heads // kv_heads
+        t = q.shape[0]
+        bf16 = q.dtype == torch.bfloat16
+        if talk.dtype != q.dtype or talk.shape[0] != (16 * -(-heads // 16) if bf16 else heads) or not talk.is_contiguous():
+            raise KernelError("talking_attention: the mixing matrix has the queries' type, padded to a multiple of 16 in bfloat16")
+        # the most keys a token can read, counted from the tile of 64 its first key lies in
+        max_keys = min(chunk + 63, shape.max_kv) if chunk else shape.max_kv
+        pitch = 64 * -(-max_keys // 64)
+        which = 0
+        if group > 16 or shape.max_q * group > 16:
+            which |= 1
+        if group <= 16 and getattr(shape, "min_q", 1) * group <= 16:
+            which |= 2
+        wide_rows, n_wide = None, 0
+        neg_q = getattr(shape, "neg_q_sorted", None)
+        if (which & 1) and neg_q is not None and getattr(shape, "rows_by_q", None) is not None:
+            n_wide = bisect.bisect_left(neg_q, -(16 // group) if group <= 16 else 0)
+            wide_rows = shape.rows_by_q
+        per_token = heads * (pitch * (4 + q.element_size()) + pitch // 64 * 8)
+        step = max(1, min(t, self.TALK_SCRATCH_BYTES // per_token))
+        n_splits, part, tickets = 1, None, None
+        if bf16 and which & 2:
+            n_splits = max(1, min(-(-2 * self.TARGET_BLOCKS // (shape.rows * kv_heads)), -(-pitch // 256), self.MAX_SPLITS))
+            if n_splits > 1:
+                part = torch.empty((shape.rows, kv_heads, n_splits, 16, head_dim), dtype=torch.float32, device=q.device)
+                tickets = self._ticket_buffer(shape.rows * kv_heads)
+        e = torch.empty((step, heads, pitch), dtype=torch.float32, device=q.device)
+        stats = torch.empty((step, heads, pitch // 64, 2), dtype=torch.float32, device=q.device)
+        w = torch.empty((step, heads, pitch), dtype=q.dtype, device=q.device)
+        for t0 in range(0, t, step):
+            self.launches += 1 + 2 * ((which & 1) + ((which >> 1) & 1)) if bf16 else 3
+            _check(lib.sb_talking_attention(
+                _p(q), q.stride(0), _p(k_cache), _p(v_cache), _p(block_table), block_table.shape[1], _p(cu_q), _p(kv_len), _p(positions),
+                heads, kv_heads, page_size, k_cache.shape[0], ctypes.c_float(scale), ctypes.c_float(float(softcap or 0.0)), int(chunk or 0),
+                _p(sinks), _p(talk), _p(e), _p(stats), _p(w), pitch, t0, min(t0 + step, t), _p(out), shape.rows, shape.max_q, max_keys, which,
+                _p(wide_rows), n_wide, n_splits, _p(part), _p(tickets), _DT[q.dtype], self._s()), "attention with mixed heads")
 
     def _tc_attention_takes(self, lib, heads, kv_heads, head_dim, page_size, window, stride) -> bool:
         key = (heads, kv_heads, head_dim, page_size, window, stride)

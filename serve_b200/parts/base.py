@@ -119,7 +119,8 @@ class Part:
         """Take the declared tensors (already on the device, in their kept dtype)."""
 
     def kernel_needs(self) -> Dict[str, Any]:
-        """Which compiled libraries this part will call: {"attention_head_dims": [...], "libraries": [names]}. The engine
+        """Which compiled libraries this part will call: {"attention_head_dims": [...], "talking_head_dims": [...] (attention with
+        mixed heads), "libraries": [names]}. The engine
         builds what all parts of a model name side by side before the first step; a part that names nothing has its
         libraries built when it first calls them."""
         return {}

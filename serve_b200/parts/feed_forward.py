@@ -1,5 +1,5 @@
 """Dense feed-forwards: gated, down( act(gate x, up x) ) with act = silu(g) * u (SwiGLU) or a clamped form, and plain,
-down( act(up x) ).
+down( act(up x) ), where act may be element by element or a polynomial of normalised powers.
 
 Reference: serve/model.py:80-85 (w1 = gate, w3 = up, w2 = down, no biases).
 Gate and up weights are fused at load into one [2*I, hidden] matrix so that one
@@ -89,10 +89,12 @@ class GatedDense(SwiGLU):
 
 @register_part("feed_forward", "plain_dense")
 class PlainDense(FeedForward):
-    """down(act(up h)) without a gate. params: hidden, intermediate, activation ("relu_squared" | "gelu_tanh" | "silu" | "tanh"),
-    names (up/down tensor names relative to prefix). The activation is computed in float32 and rounded once."""
+    """down(act(up h)) without a gate. params: hidden, intermediate, activation ("relu_squared" | "gelu_tanh" | "silu" | "tanh" |
+    "poly_norm"), eps (poly_norm), names (up/down/act tensor names relative to prefix). The activation is computed in float32 and
+    rounded once. poly_norm: a N(z) + b N(z^2) + c N(z^3) + e with a learned [a, b, c, e] ("act"), powers element by element, N(u) =
+    u / sqrt(mean(u^2) + eps) over a token's ``intermediate`` values."""
 
-    ACTIVATIONS = ("relu_squared", "gelu_tanh", "silu", "tanh")
+    ACTIVATIONS = ("relu_squared", "gelu_tanh", "silu", "tanh", "poly_norm")
 
     def __init__(self, spec, runtime):
         super().__init__(spec, runtime)
@@ -103,21 +105,31 @@ class PlainDense(FeedForward):
             raise ValueError(f"plain_dense: activation {self.activation!r} is not known ({', '.join(self.ACTIVATIONS)})")
         names = p.get("names", {})
         self.up_name, self.down_name = self.prefix + names.get("up", "up"), self.prefix + names.get("down", "down")
-        self.w_up = self.w_down = None
+        self.poly = self.activation == "poly_norm"
+        self.act_name = self.prefix + names.get("act", "act")
+        self.eps = float(p["eps"]) if self.poly else 0.0
+        self.w_up = self.w_down = self.coef = None
 
     def kernel_needs(self):
         return {"libraries": ["prep"]}
 
     def tensor_decls(self):
-        return [TensorDecl(self.up_name, (self.intermediate, self.hidden)), TensorDecl(self.down_name, (self.hidden, self.intermediate))]
+        decls = [TensorDecl(self.up_name, (self.intermediate, self.hidden)), TensorDecl(self.down_name, (self.hidden, self.intermediate))]
+        return decls + ([TensorDecl(self.act_name, (4,), role="vector", init="norm")] if self.poly else [])
 
     def load(self, tensors):
         self.w_up, self.w_down = tensors[self.up_name].contiguous(), tensors[self.down_name].contiguous()
+        if self.poly:
+            self.coef = tensors[self.act_name].float().contiguous()
 
     def forward(self, h, ctx):
         rt = self.rt
         act = rt.empty_act((h.shape[0], self.intermediate))
-        rt.kernels.linear_activation(h, self.w_up, act, self.activation)
+        if self.poly:
+            rt.kernels.linear(h, self.w_up, act)
+            rt.kernels.poly_norm(act, self.coef, self.eps, act)
+        else:
+            rt.kernels.linear_activation(h, self.w_up, act, self.activation)
         out = rt.empty_act((h.shape[0], self.hidden))
         rt.kernels.linear(act, self.w_down, out)
         return out

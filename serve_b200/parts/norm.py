@@ -1,4 +1,4 @@
-"""RMS normalisation and layer normalisation, each fused with the residual addition that precedes it.
+"""RMS normalisation (of the whole row or of parts of it) and layer normalisation, each fused with the residual addition that precedes it.
 
 Reference formula (serve/model.py:63-68): y = x32 * rsqrt(mean(x32^2) + eps),
 cast to the model dtype, times weight. Here the residual stream itself is kept
@@ -73,6 +73,66 @@ class LayerNorm(RMSNorm):
     def forward_rows(self, x, delta, rows, ctx):
         out = self.rt.empty_act((rows.shape[0], self.size))
         self.rt.kernels.add_layernorm_rows(x, self._delta(delta), rows, self.weight, self.eps, out)
+        return out
+
+
+@register_part("norm", "grouped_rms")
+class GroupedRMSNorm(Norm):
+    """The vector is cut into ``groups`` equal consecutive parts, each divided by its own sqrt(mean(part^2) + eps); then a weight
+    per element. ``scale_name``: a second factor per element (a layer scale behind a norm after a sub-layer), multiplied into the
+    weight at load in float. The same fusion with the residual addition as the other norms; and the norm of the sub-layer before
+    (a ``DeferredNorm`` of this kind with the same parts) is applied in the same kernel: x += n'(a); y = n(x).
+    params: size, groups, eps, weight_name, scale_name."""
+
+    def __init__(self, spec, runtime):
+        super().__init__(spec, runtime)
+        p = spec.params
+        self.size, self.groups, self.eps = int(p["size"]), int(p.get("groups") or 1), float(p["eps"])
+        if self.size % self.groups:
+            raise ValueError(f"grouped_rms: {self.size} elements cannot be cut into {self.groups} equal parts")
+        self.weight_name = self.prefix + p.get("weight_name", "weight")
+        self.scale_name = self.prefix + p["scale_name"] if p.get("scale_name") else None
+        self.weight = None
+
+    def kernel_needs(self):
+        return {"libraries": ["prep"]}
+
+    def tensor_decls(self):
+        names = [self.weight_name] + ([self.scale_name] if self.scale_name else [])
+        return [TensorDecl(n, (self.size,), role="vector", init="norm") for n in names]
+
+    def load(self, tensors):
+        w = tensors[self.weight_name].float()
+        if self.scale_name:
+            w = w * tensors[self.scale_name].float()
+        self.weight = w.contiguous()
+
+    def _split(self, delta):
+        """(tensor to add or None, the weight of the norm it goes through first or None)."""
+        if isinstance(delta, DeferredNorm):
+            n = delta.norm
+            if isinstance(n, GroupedRMSNorm) and (n.size, n.groups, n.eps) == (self.size, self.groups, self.eps):
+                return delta.a, n.weight
+            return delta.plain(), None
+        return plain_delta(delta), None
+
+    def forward(self, x, delta, ctx):
+        out = self.rt.empty_act((x.shape[0], self.size))
+        a, through = self._split(delta)
+        self.rt.kernels.add_grouped_rmsnorm(x, a, through, None, self.weight, self.groups, self.eps, out)
+        return out
+
+    def forward_rows(self, x, delta, rows, ctx):
+        out = self.rt.empty_act((rows.shape[0], self.size))
+        a, through = self._split(delta)
+        self.rt.kernels.add_grouped_rmsnorm(x, a, through, rows, self.weight, self.groups, self.eps, out)
+        return out
+
+    def apply(self, a):
+        import torch
+
+        out = torch.empty((a.shape[0], self.size), dtype=torch.float32, device=a.device)
+        self.rt.kernels.add_grouped_rmsnorm(None, a, None, None, self.weight, self.groups, self.eps, out)
         return out
 
 

@@ -225,18 +225,22 @@ class EmuKernels:
         x.add_(bias.to(x.dtype))
 
     def qk_prepare(self, sums, bias, positions, token_row, heads, kv_heads, head_dim, dim, q_weight, k_weight, eps, inv_freq, rot_dims,
-                   q_out, k_cache, v_cache, block_table, page_size, head_norm=False):
+                   q_out, k_cache, v_cache, block_table, page_size, head_norm=False, keys_are_values=False):
         t, d, m = sums.shape[0], head_dim, self.math
-        x = sums[:, : (heads + 2 * kv_heads) * d].to(m)      # (the row may go on with columns that are not the kernel's)
+        n = heads + (1 if keys_are_values else 2) * kv_heads
+        x = sums[:, : n * d].to(m)                           # (the row may go on with columns that are not the kernel's)
         if bias is not None:
             x = x + bias.to(m)
-        x = x.reshape(t, heads + 2 * kv_heads, d)
+        x = x.reshape(t, n, d)
         ang = positions.to(torch.float32)[:, None] * inv_freq.to(torch.float32)[None, : rot_dims // 2]
         cos, sin = ang.cos().to(m)[:, None, :], ang.sin().to(m)[:, None, :]
 
         def prepare(v, n_heads, weight):
             v = v.reshape(t, n_heads * d)
-            if weight is not None:
+            if head_norm == "before":
+                v = v.view(t, n_heads, d)
+                v = v * torch.rsqrt(v.pow(2).sum(-1, keepdim=True) / dim + eps) * weight.to(m)
+            elif weight is not None:
                 v = v * torch.rsqrt(v.pow(2).sum(-1, keepdim=True) / (n_heads * dim) + eps) * weight.to(m)
             v = v.view(t, n_heads, d).clone()
             half = rot_dims // 2
@@ -244,14 +248,69 @@ class EmuKernels:
                 a, b = v[..., :half].clone(), v[..., half: rot_dims].clone()
                 v[..., :half] = a * cos - b * sin
                 v[..., half: rot_dims] = b * cos + a * sin
-            if head_norm:
+            if head_norm is True:
                 v = v * torch.rsqrt(v.pow(2).sum(-1, keepdim=True) / dim + eps)
             return v
 
         q_out.copy_(prepare(x[:, :heads], heads, q_weight).reshape(t, heads * d).to(q_out.dtype))
         if kv_heads:
             self._write_pages(k_cache, prepare(x[:, heads: heads + kv_heads], kv_heads, k_weight), positions, token_row, block_table, page_size)
-            self._write_pages(v_cache, x[:, heads + kv_heads:], positions, token_row, block_table, page_size)
+            self._write_pages(v_cache, x[:, n - kv_heads:], positions, token_row, block_table, page_size)
+
+    def add_grouped_rmsnorm(self, x, delta, through, rows, weight, groups, eps, out):
+        def norm(v, w):
+            v = v.to(self.math)
+            parts = v.reshape(v.shape[0], groups, v.shape[1] // groups)
+            return (parts * torch.rsqrt(parts.pow(2).mean(-1, keepdim=True) + eps)).reshape(v.shape) * w.to(self.math)
+
+        d = None if delta is None else (norm(delta, through).to(torch.float32) if through is not None else delta.to(torch.float32))
+        if x is None:
+            out.copy_(norm(d, weight).to(out.dtype))
+        elif rows is not None:
+            v = x[rows.long()] if d is None else x[rows.long()] + d[rows.long()]
+            out.copy_(norm(v, weight).to(out.dtype))
+        else:
+            if d is not None:
+                x.add_(d)
+            out.copy_(norm(x, weight).to(out.dtype))
+
+    def poly_norm(self, z, coef, eps, out):
+        v = z.to(self.math)
+        a, b, c, e = coef.to(self.math).unbind()
+        unit = lambda u: u * torch.rsqrt(u.pow(2).mean(-1, keepdim=True) + eps)
+        out.copy_((a * unit(v) + b * unit(v * v) + c * unit(v * v * v) + e).to(out.dtype))
+
+    def talking_attention(self, q, k_cache, v_cache, block_table, cu_q, kv_len, positions, heads, kv_heads, head_dim, page_size, scale, talk,
+                          out, shape, chunk=0, softcap=0.0, sinks=None):
+        d, g, m = head_dim, heads // kv_heads, self.math
+        mix = talk[:heads, :heads].to(m)
+        cu, lens = cu_q.tolist(), kv_len.tolist()
+        for r in range(len(lens)):
+            q0, q1, L = cu[r], cu[r + 1], lens[r]
+            n = q1 - q0
+            if n == 0:
+                continue
+            lo = ((L - n) // chunk) * chunk if chunk else 0
+            keys = torch.arange(lo, L, device=q.device)
+            pages = block_table[r].long()[keys // page_size]
+            assert bool((pages >= 0).all()), "attention reads a missing page"
+            k = k_cache[pages, :, keys % page_size].to(m).repeat_interleave(g, 1)
+            v = v_cache[pages, :, keys % page_size].to(m).repeat_interleave(g, 1)
+            s = torch.einsum("thd,shd->hts", q[q0:q1, : heads * d].view(n, heads, d).to(m), k) * scale
+            if softcap:
+                s = softcap * torch.tanh(s / softcap)
+            qp, kp = torch.arange(L - n, L, device=q.device)[:, None], keys[None, :]
+            mask = kp > qp
+            if chunk:
+                mask = mask | (kp < (qp // chunk) * chunk)
+            s = s.masked_fill(mask[None], float("-inf"))
+            if sinks is not None:
+                s = torch.cat([s, sinks.to(m)[:, None, None].expand(heads, n, 1)], -1)
+                p = torch.softmax(s, -1)[..., :-1]
+            else:
+                p = torch.softmax(s, -1)
+            p = torch.einsum("hg,gts->hts", mix, p)
+            out[q0:q1] = torch.einsum("hts,shd->thd", p, v).reshape(n, heads * d).to(out.dtype)
 
     def linear_batched(self, a, w, out):
         """out[:, b] = a[:, b] @ w[b]^T for every b: a [M, B, K], w [B, N, K], out [M, B, N] (views with any row strides)."""
