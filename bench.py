@@ -11,8 +11,8 @@ of three: the way the reference's own benchmark times its generate()); ``prefill
 compares the decode step with the bytes it has to read (every weight once, and the cache of the live requests).
 The weights (2.47 GB) are larger than the L2 cache, so no flush is needed between steps.
 
-``--design rogisun`` (or ``bapavik``, ``lilunex``, ``gebilorn``) is another measurement altogether and leaves the line above as it is: prefill and decode
-throughput of the Rogisun decoder (three layers, one of each mixer, routed experts) at layer sizes of real models,
+``--design rogisun`` (or ``bapavik``, ``lilunex``, ``gebilorn``, ``vivepel``) is another measurement altogether and leaves the line above as it
+is: prefill and decode throughput of the Rogisun decoder (three layers, one of each mixer, routed experts) at layer sizes of real models,
 beside a Llama decoder of equal width, depth and active feed-forward size, each with the device time of every kernel
 of one prompt step and one decoding step; it prints its own JSON line (see design_bench).
 
@@ -407,7 +407,21 @@ def gebilorn_at(width: int, vocab: int = 32000):
                              "max_position": CONTEXT})
 
 
-DESIGNS = {"rogisun": rogisun_at, "bapavik": bapavik_at, "lilunex": lilunex_at, "gebilorn": gebilorn_at}
+def vivepel_at(width: int, vocab: int = 32000):
+    """A Vivepel configuration with layers of a real model's sizes: attention with mixed heads of 128 (half of a head rotated, blocks
+    of 1,024 positions, capped scores) and a dense feed-forward with as many weights as the Llama decoder's gated one; norms over
+    eight parts of the row."""
+    from serve_b200.config import config_from_dict
+
+    heads, _experts, top, ff = DESIGN_SIZES[str(width)]
+    att = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 0.08, "softcap": 30.0, "mask": {"size": 1024},
+           "rot": {"base": 500000.0, "dims": 64}}
+    layers = [{"type": "attention", "mixer": att, "mlp": {"kind": "dense", "ff": 3 * top * ff // 2}}] * 3
+    return config_from_dict({"architecture": "Vivepel", "width": width, "vocab": vocab, "norm": {"eps": 1e-5, "groups": 8}, "layers": layers,
+                             "max_position": CONTEXT})
+
+
+DESIGNS = {"rogisun": rogisun_at, "bapavik": bapavik_at, "lilunex": lilunex_at, "gebilorn": gebilorn_at, "vivepel": vivepel_at}
 
 
 def kernel_times(eng, entries, end):
@@ -454,7 +468,7 @@ def prefill_many(eng, vocab, requests, each, reps=5, seed=11):
 
 def design_bench(args):
     """Prefill (one prompt of 2,048 tokens) and decode (batch 8 after 2,048-token prompts, from CUDA graphs) of the named design
-    (Rogisun, Bapavik, Lilunex or Gebilorn) and of the Llama decoder of equal size, at each width asked for, bfloat16, random weights; CUDA events on the stream, the
+    (Rogisun, Bapavik, Lilunex, Gebilorn or Vivepel) and of the Llama decoder of equal size, at each width asked for, bfloat16, random weights; CUDA events on the stream, the
     weights alone exceed the L2 cache. Prints one JSON line: per width and design the two rates, the rate of a step of 8 prompts
     of 256 tokens (the same tokens side by side: what a recurrence walks in turn for one prompt it walks at once for eight),
     and the kernels of one prompt step and one (eager) decoding step with their device times."""
