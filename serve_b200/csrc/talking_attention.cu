@@ -18,23 +18,22 @@
 // bfloat16 numbers (p = hi + lo to 2^-17), so the mixed weights keep float's sums and are rounded once, for the product with the
 // values. In float32 everything is plain fused multiply-adds. Two shapes, as in the other attention kernels: requests with at most
 // 16 rows (tokens x heads of a kv head) are "deep", the others "wide". Compile with -DSB_HEAD_DIM=<multiple of 16, 16..256>.
-#include "common.cuh"
+#include "talking_attention.cuh"
 
 #ifndef SB_HEAD_DIM
 #error "define SB_HEAD_DIM"
 #endif
 
 using namespace sb;
+using namespace talk;
 typedef __nv_bfloat16 bf16;
 
 namespace {
 
 constexpr int D = SB_HEAD_DIM;
-constexpr int BN = 64;               // keys per tile
 constexpr int LDS = D + 8;           // row stride of a key or value tile in shared memory (elements)
 constexpr int LDW = BN + 8;          // row stride of a weight tile in shared memory
 constexpr int CHUNKS = D / 8;        // 16-byte pieces per row
-constexpr float LOG2E = 1.4426950408889634f;
 static_assert(D % 16 == 0 && D >= 16 && D <= 256, "head_dim must be a multiple of 16 in 16..256");
 
 __device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -60,30 +59,6 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
   return *reinterpret_cast<uint32_t*>(&v);
 }
-__device__ __forceinline__ float ex2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-
-struct Params {
-  const void* q; int q_stride;
-  const void* kc; const void* vc;
-  const int* block_table; int bt_width;
-  const int* cu_q; const int* kv_len; const int* positions;
-  int H, G, per, ps, ps_shift, num_pages;    // query heads, kv heads, query heads of a kv head; page size (its log2, or -1)
-  float scale, cap, cap_in;                  // cap 0: none; cap_in = scale / cap
-  int chunk;
-  const float* sinks;                        // [H] or null
-  const void* talk;                          // [Hp, Hp] (bfloat16, zeros beyond H) or [H, H] (float32), row = output head
-  float* e; float2* stats; void* w;          // scratch: [tokens, H, pitch] floats, [tokens, H, pitch / 64], [tokens, H, pitch]
-  int pitch, t_lo, t_hi;                     // the launch covers tokens [t_lo, t_hi) of the step
-  void* out;                                 // [T, H * D]
-  const int* wide_rows; int deep_on;         // requests the wide shape covers (null: all); deep_on: the deep shape takes the small ones
-  int n_splits; float* part; int* tickets;   // values, deep: key splits, [R, G, splits, 16, D] floats, [R, G] zeros
-};
-
-__device__ __forceinline__ int first_key(const Params& p, int pos) { return p.chunk > 0 ? (pos / p.chunk) * p.chunk : 0; }
 
 // Where key ``key`` of kv head hk lies in a cache tensor (elements), or -1 where there is no page.
 __device__ __forceinline__ long long cache_row(const Params& p, const int* bt, int hk, int key) {
@@ -106,16 +81,10 @@ __device__ __forceinline__ void load_tile(const Params& p, const bf16* cache, co
   }
 }
 
-// A raw product as a score in units of log2: scaled, capped. tanh(z) = 1 - 2 / (1 + e^(2z)); its error is about 2^-23 of the cap.
-__device__ __forceinline__ float score_log2(const Params& p, float raw) {
-  if (p.cap > 0.f) return (p.cap * LOG2E) * (1.f - __fdividef(2.f, 1.f + ex2(raw * p.cap_in * (2.f * LOG2E))));
-  return raw * p.scale * LOG2E;
-}
-
 // A row's scores of one tile (16 a lane over a quad of lanes, keys kt + 16 i + 4 tq + 0..3) -> e and the tile's (m, sum).
 // raw[i][0..3]: the products; the row stores its tile if it reads any of its keys.
 __device__ __forceinline__ void finish_row(const Params& p, float (&raw)[4][4], int kt, int first, int pos, size_t row, int tq) {
-  float m = -INFINITY;
+  float m = p.fixed ? 0.f : -INFINITY;
 #pragma unroll
   for (int i = 0; i < 4; ++i)
 #pragma unroll
@@ -123,10 +92,12 @@ __device__ __forceinline__ void finish_row(const Params& p, float (&raw)[4][4], 
       const int key = kt + 16 * i + 4 * tq + c;
       const float s = (key >= first && key <= pos) ? score_log2(p, raw[i][c]) : -INFINITY;
       raw[i][c] = s;
-      m = fmaxf(m, s);
+      if (!p.fixed) m = fmaxf(m, s);
     }
-  m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, 1));
-  m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, 2));
+  if (!p.fixed) {
+    m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, 1));
+    m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, 2));
+  }
   const int base = first & ~(BN - 1);
   const bool live = pos >= 0 && kt >= base && kt <= pos;      // (then at least one key of the tile is visible and m is finite)
   float sum = 0.f;
@@ -334,27 +305,36 @@ __global__ void __launch_bounds__(128) scores_deep_kernel(const Params p) {
 }
 
 // ---------------------------------------------------------------------------------------------------------- mix
-// Every head's maximum (log2) and 1 / denominator of token row t (scratch), from the tiles' statistics: one warp a head at a time.
+// Every head's maximum (log2) and 1 / denominator of token row t (scratch), from the tiles' statistics: ``team`` neighbouring
+// threads a head (a power of two up to 32).
 __device__ __forceinline__ void token_softmax(const Params& p, int t, int n_tiles, float* M_s, float* inv_s) {
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
   const int tiles_pitch = p.pitch / BN;
-  for (int h = warp; h < p.H; h += n_warps) {
-    const float2* st = p.stats + ((size_t)t * p.H + h) * tiles_pitch;
-    float m = p.sinks ? p.sinks[h] * LOG2E : -INFINITY;
-    for (int i = lane; i < n_tiles; i += 32) m = fmaxf(m, st[i].x);
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
-    float l = 0.f;
-    for (int i = lane; i < n_tiles; i += 32) l += st[i].y * exp2f(st[i].x - m);
-    l = warp_sum(l);
-    if (p.sinks) l += exp2f(p.sinks[h] * LOG2E - m);
-    if (lane == 0) { M_s[h] = m; inv_s[h] = 1.f / l; }
+  int team = 32;
+  while (team > 1 && team * p.H > (int)blockDim.x) team >>= 1;
+  const int at = threadIdx.x & (team - 1), per_round = blockDim.x / team;
+  const int rounds = (p.H + per_round - 1) / per_round;
+  for (int k = 0; k < rounds; ++k) {
+    const int h = k * per_round + threadIdx.x / team;
+    const bool ok = h < p.H;
+    const float2* st = p.stats + ((size_t)t * p.H + (ok ? h : 0)) * tiles_pitch;
+    const float sink = (p.sinks && ok) ? p.sinks[h] * LOG2E : -INFINITY;
+    float m = p.fixed ? 0.f : sink, l = 0.f;
+    if (p.fixed) {
+      for (int i = at; i < n_tiles; i += team) l += st[i].y;
+    } else {
+      for (int i = at; i < n_tiles; i += team) m = fmaxf(m, st[i].x);
+      for (int o = team >> 1; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+      for (int i = at; i < n_tiles; i += team) l += st[i].y * exp2f(st[i].x - m);
+    }
+    for (int o = team >> 1; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
+    if (ok && at == 0) { M_s[h] = m; inv_s[h] = 1.f / (l + exp2f(sink - m)); }
   }
   __syncthreads();
 }
 
-// grid (tokens, strip blocks), 4 warps; a warp takes strips of 32 keys. The product is talk [16 MT x Hp] times p [Hp x 32 keys];
-// column n of the q-th of four product tiles stands for key 4 n + q, so a lane reads 16 bytes of a head's row and writes 16.
+// grid (tokens, tile blocks), 4 warps; a warp takes tiles of 64 keys, two strips of 32 at a time. The product is talk [16 MT x Hp]
+// times p [Hp x 32 keys]; column n of the q-th of a strip's four product tiles stands for key 4 n + q, so a lane reads 16 bytes of a
+// head's row and writes 16.
 template <int MT>
 __global__ void __launch_bounds__(128) mix_kernel(const Params p) {
   extern __shared__ float mix_s[];
@@ -362,74 +342,90 @@ __global__ void __launch_bounds__(128) mix_kernel(const Params p) {
   pdl_wait();
   const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, tq = lane & 3;
   const int pos = p.positions[p.t_lo + t];
-  const int base = first_key(p, pos) & ~(BN - 1), n_tiles = (pos - base) / BN + 1, n_strips = 2 * n_tiles;
-  if ((int)blockIdx.y * 4 >= n_strips) return;
+  const int base = first_key(p, pos) & ~(BN - 1), n_tiles = (pos - base) / BN + 1;
+  const int n_all = p.zero_ahead ? min((pos + p.zero_ahead - base) / BN + 1, p.pitch / BN) : n_tiles;
+  if ((int)blockIdx.y * 4 >= n_all) return;
+  const int tiles_pitch = p.pitch / BN;
   token_softmax(p, t, n_tiles, M_s, inv_s);
   const int kt_n = (p.H + 15) / 16, hp = kt_n * 16;
   const uint32_t* talk = reinterpret_cast<const uint32_t*>(p.talk);     // pairs of neighbouring columns
   const size_t row0 = (size_t)t * p.H;
-  for (int strip = blockIdx.y * 4 + warp; strip < n_strips; strip += gridDim.y * 4) {
+  for (int tile = blockIdx.y * 4 + warp; tile < n_all; tile += gridDim.y * 4) {
+    if (tile >= n_tiles) {
+      for (int h = g; h < p.H; h += 8) {
+        uint4* dst = reinterpret_cast<uint4*>((bf16*)p.w + (row0 + h) * p.pitch + tile * BN + tq * 16);
+        dst[0] = dst[1] = make_uint4(0, 0, 0, 0);
+      }
+      continue;
+    }
     for (int mg = 0; mg < kt_n; mg += MT) {
-      float acc[MT][4][4];
+      float acc[2][MT][4][4];
 #pragma unroll
-      for (int m = 0; m < MT; ++m)
+      for (int s = 0; s < 2; ++s)
 #pragma unroll
-        for (int n = 0; n < 4; ++n) acc[m][n][0] = acc[m][n][1] = acc[m][n][2] = acc[m][n][3] = 0.f;
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+          for (int n = 0; n < 4; ++n) acc[s][m][n][0] = acc[s][m][n][1] = acc[s][m][n][2] = acc[s][m][n][3] = 0.f;
       for (int kk = 0; kk < kt_n; ++kk) {
-        // heads kk * 16 + 2 tq + {0, 1, 8, 9}: p of four keys each
-        float pv[4][4];
+        // heads kk * 16 + 2 tq + {0, 1, 8, 9}: e of four keys each, of both strips
+        float4 ev[2][4];
+        float f[4];
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
           const int h = kk * 16 + 2 * tq + (i & 1) + ((i >> 1) << 3);
-          float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-          if (h < p.H) {
-            v = *reinterpret_cast<const float4*>(p.e + (row0 + h) * p.pitch + strip * 32 + g * 4);
-            const float f = ex2(p.stats[(row0 + h) * (p.pitch / BN) + (strip >> 1)].x - M_s[h]) * inv_s[h];
-            v.x *= f; v.y *= f; v.z *= f; v.w *= f;
-          }
-          pv[i][0] = v.x; pv[i][1] = v.y; pv[i][2] = v.z; pv[i][3] = v.w;
+          const float* src = p.e + (row0 + h) * p.pitch + tile * BN + g * 4;
+          ev[0][i] = h < p.H ? __ldcs(reinterpret_cast<const float4*>(src)) : make_float4(0.f, 0.f, 0.f, 0.f);
+          ev[1][i] = h < p.H ? __ldcs(reinterpret_cast<const float4*>(src + 32)) : make_float4(0.f, 0.f, 0.f, 0.f);
+          f[i] = h < p.H ? inv_s[h] : 0.f;
+          if (!p.fixed && h < p.H) f[i] *= ex2(p.stats[(row0 + h) * tiles_pitch + tile].x - M_s[h]);
         }
-        uint32_t hi[4][2], lo[4][2];
 #pragma unroll
-        for (int n = 0; n < 4; ++n)
+        for (int s = 0; s < 2; ++s) {
+          uint32_t hi[4][2], lo[4][2];
 #pragma unroll
           for (int j = 0; j < 2; ++j) {
-            const float x = pv[2 * j][n], y = pv[2 * j + 1][n];
-            const __nv_bfloat162 h2 = __floats2bfloat162_rn(x, y);
-            hi[n][j] = *reinterpret_cast<const uint32_t*>(&h2);
-            lo[n][j] = pack_bf16(x - __low2float(h2), y - __high2float(h2));
-          }
-#pragma unroll
-        for (int m = 0; m < MT; ++m) {
-          if (mg + m < kt_n) {
-            const uint32_t* a = talk + ((size_t)((mg + m) * 16 + g) * hp + kk * 16) / 2 + tq;
-            const uint32_t a0 = __ldg(a), a1 = __ldg(a + 4 * hp), a2 = __ldg(a + 4), a3 = __ldg(a + 4 * hp + 4);
+            const float4 a = ev[s][2 * j], b = ev[s][2 * j + 1];
+            const float fa = f[2 * j], fb = f[2 * j + 1];
+            const float xs[4] = {a.x * fa, a.y * fa, a.z * fa, a.w * fa}, ys[4] = {b.x * fb, b.y * fb, b.z * fb, b.w * fb};
 #pragma unroll
             for (int n = 0; n < 4; ++n) {
-              mma_bf16(acc[m][n], a0, a1, a2, a3, lo[n][0], lo[n][1]);
-              mma_bf16(acc[m][n], a0, a1, a2, a3, hi[n][0], hi[n][1]);
+              const __nv_bfloat162 h2 = __floats2bfloat162_rn(xs[n], ys[n]);
+              hi[n][j] = *reinterpret_cast<const uint32_t*>(&h2);
+              lo[n][j] = pack_bf16(xs[n] - __low2float(h2), ys[n] - __high2float(h2));
+            }
+          }
+#pragma unroll
+          for (int m = 0; m < MT; ++m) {
+            if (mg + m < kt_n) {
+              const uint32_t* a = talk + ((size_t)((mg + m) * 16 + g) * hp + kk * 16) / 2 + tq;
+              const uint32_t a0 = __ldg(a), a1 = __ldg(a + 4 * hp), a2 = __ldg(a + 4), a3 = __ldg(a + 4 * hp + 4);
+#pragma unroll
+              for (int n = 0; n < 4; ++n) {
+                mma_bf16(acc[s][m][n], a0, a1, a2, a3, lo[n][0], lo[n][1]);
+                mma_bf16(acc[s][m][n], a0, a1, a2, a3, hi[n][0], hi[n][1]);
+              }
             }
           }
         }
       }
 #pragma unroll
-      for (int m = 0; m < MT; ++m) {
+      for (int s = 0; s < 2; ++s)
 #pragma unroll
-        for (int half = 0; half < 2; ++half) {
-          const int h = (mg + m) * 16 + g + 8 * half;
-          if (h < p.H) {
-            uint4 v;
-            v.x = pack_bf16(acc[m][0][2 * half], acc[m][1][2 * half]);
-            v.y = pack_bf16(acc[m][2][2 * half], acc[m][3][2 * half]);
-            v.z = pack_bf16(acc[m][0][2 * half + 1], acc[m][1][2 * half + 1]);
-            v.w = pack_bf16(acc[m][2][2 * half + 1], acc[m][3][2 * half + 1]);
-            *reinterpret_cast<uint4*>((bf16*)p.w + (row0 + h) * p.pitch + strip * 32 + tq * 8) = v;
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+          for (int half = 0; half < 2; ++half) {
+            const int h = (mg + m) * 16 + g + 8 * half;
+            if (h < p.H) {
+              uint4 v;
+              v.x = pack_bf16(acc[s][m][0][2 * half], acc[s][m][1][2 * half]);
+              v.y = pack_bf16(acc[s][m][2][2 * half], acc[s][m][3][2 * half]);
+              v.z = pack_bf16(acc[s][m][0][2 * half + 1], acc[s][m][1][2 * half + 1]);
+              v.w = pack_bf16(acc[s][m][2][2 * half + 1], acc[s][m][3][2 * half + 1]);
+              *reinterpret_cast<uint4*>((bf16*)p.w + (row0 + h) * p.pitch + tile * BN + s * 32 + tq * 8) = v;
+            }
           }
-        }
-      }
     }
   }
-  pdl_launch_dependents();
 }
 
 // float32: a block per (token, tile of 64 keys); the tile's weights of all heads in shared memory (in parts of 128 heads).
@@ -741,12 +737,14 @@ template <typename K> int allow_smem(K k, size_t bytes) {
 // buffers for t_hi - t_lo tokens of ``pitch`` keys (a multiple of 64 no shorter than what any of them reads, counted from its base);
 // out [T, H * D]. which: bit 0 wide requests, bit 1 deep ones (float32 has one shape). wide_rows [n_wide] or null (all R).
 // n_splits > 1: part [R, G, n_splits, 16, D] floats and tickets [R, G], zero before and after. max_keys: the most keys (from its
-// base) a token of the launch reads, max_q the most tokens a request brings: they size grids only.
+// base) a token of the launch reads, max_q the most tokens a request brings: they size grids only. use_tc: wide requests may run on
+// tcgen05 (q has n_tokens rows; *error is raised if a bounded wait runs out).
 SB_EXPORT int sb_talking_attention(const void* q, int q_stride, const void* kc, const void* vc, const int* block_table, int bt_width,
                                    const int* cu_q, const int* kv_len, const int* positions, int H, int G, int ps, int num_pages, float scale,
                                    float softcap, int chunk, const float* sinks, const void* talk, float* e, void* stats, void* w, int pitch,
                                    int t_lo, int t_hi, void* out, int R, int max_q, int max_keys, int which, const int* wide_rows, int n_wide,
-                                   int n_splits, float* part, int* tickets, int dtype, cudaStream_t stream) {
+                                   int n_splits, float* part, int* tickets, int n_tokens, int* error, int use_tc, int dtype,
+                                   cudaStream_t stream) {
   const int n_tok = t_hi - t_lo;
   if (n_tok <= 0 || R <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G || ps <= 0 || bt_width <= 0 || pitch <= 0 || pitch % BN || max_keys > pitch || q_stride < H * D || !talk || !e ||
@@ -761,6 +759,8 @@ SB_EXPORT int sb_talking_attention(const void* q, int q_stride, const void* kc, 
   p.ps_shift = -1;
   for (int s = 0; s < 30; ++s) if ((1 << s) == ps) p.ps_shift = s;
   p.scale = scale; p.cap = softcap > 0.f ? softcap : 0.f; p.cap_in = softcap > 0.f ? scale / softcap : 0.f;
+  p.fixed = softcap > 0.f && softcap <= FIXED_CAP && dtype == SB_DTYPE_BF16;
+  p.zero_ahead = 0;
   p.chunk = chunk; p.sinks = sinks; p.talk = talk; p.e = e; p.stats = (float2*)stats; p.w = w; p.pitch = pitch; p.t_lo = t_lo; p.t_hi = t_hi;
   p.out = out; p.wide_rows = wide_rows; p.deep_on = (which & 2) != 0; p.n_splits = n_splits; p.part = part; p.tickets = tickets;
   const int max_tiles = (max_keys + BN - 1) / BN;
@@ -786,21 +786,27 @@ SB_EXPORT int sb_talking_attention(const void* q, int q_stride, const void* kc, 
   const int nz = wide_rows ? n_wide : R;
   const bool wide = (which & 1) && nz > 0, deep = (which & 2) != 0;
   const dim3 wgrid(G, (unsigned)((max_q * p.per + 16 * NW - 1) / (16 * NW)), (unsigned)max(nz, 1));
-  if (wide) {
+  const bool tc = wide && use_tc && error && tc_takes(H, G, ps, q_stride, chunk);
+  if (tc) {
+    p.zero_ahead = tc_tokens_per_tile(H, G) - 1;
+    if (int rc = tc_scores(p, n_tokens, max_keys, max_q, nz, error, stream)) return rc;
+  } else if (wide) {
     const size_t smem = (size_t)(16 * NW + 2 * BN) * LDS * sizeof(bf16);
     if (int rc = allow_smem(scores_wide_kernel<NW>, smem)) return rc;
     SB_PDL_CHECK(launch_pdl(scores_wide_kernel<NW>, wgrid, dim3(NW * 32), smem, stream, p));
   }
   if (deep) SB_PDL_CHECK(launch_pdl(scores_deep_kernel, dim3(G, (unsigned)((max_tiles + 3) / 4), R), dim3(128), 0, stream, p));
   {
-    // few tokens: strips go to blocks of their own; many: a block walks its token's strips
-    const int want = (4 * sm_count() + n_tok - 1) / n_tok, have = (2 * max_tiles + 3) / 4;
+    // few tokens: tiles go to blocks of their own; many: a block walks its token's tiles
+    const int want = (4 * sm_count() + n_tok - 1) / n_tok, have = (max_tiles + 3) / 4;
     const dim3 grid(n_tok, (unsigned)max(1, min(want, have)));
     if (H <= 16) SB_PDL_CHECK(launch_pdl(mix_kernel<1>, grid, dim3(128), mix_smem, stream, p));
     else if (H <= 32) SB_PDL_CHECK(launch_pdl(mix_kernel<2>, grid, dim3(128), mix_smem, stream, p));
     else SB_PDL_CHECK(launch_pdl(mix_kernel<4>, grid, dim3(128), mix_smem, stream, p));
   }
-  if (wide) {
+  if (tc) {
+    if (int rc = tc_values(p, max_q, nz, error, stream)) return rc;
+  } else if (wide) {
     const size_t smem = (size_t)2 * (16 * NW * LDW + BN * LDS) * sizeof(bf16);
     if (int rc = allow_smem(values_wide_kernel<NW>, smem)) return rc;
     SB_PDL_CHECK(launch_pdl(values_wide_kernel<NW>, wgrid, dim3(NW * 32), smem, stream, p));

@@ -93,7 +93,7 @@ def attention_job(head_dim: int):
 
 def talking_attention_job(head_dim: int):
     """Attention whose heads' weights are mixed before the values (built when a model first asks for it)."""
-    return {"name": f"sb_talk_hd{head_dim}", "sources": ["talking_attention.cu"], "defines": [f"SB_HEAD_DIM={head_dim}"]}
+    return {"name": f"sb_talk_hd{head_dim}", "sources": ["talking_attention.cu", "talking_attention_tc.cu"], "defines": [f"SB_HEAD_DIM={head_dim}"]}
 
 
 def layer_run_job(head_dim: int):
@@ -812,7 +812,8 @@ class CudaKernels:
                 _p(q), q.stride(0), _p(k_cache), _p(v_cache), _p(block_table), block_table.shape[1], _p(cu_q), _p(kv_len), _p(positions),
                 heads, kv_heads, page_size, k_cache.shape[0], ctypes.c_float(scale), ctypes.c_float(float(softcap or 0.0)), int(chunk or 0),
                 _p(sinks), _p(talk), _p(e), _p(stats), _p(w), pitch, t0, min(t0 + step, t), _p(out), shape.rows, shape.max_q, max_keys, which,
-                _p(wide_rows), n_wide, n_splits, _p(part), _p(tickets), _DT[q.dtype], self._s()), "attention with mixed heads")
+                _p(wide_rows), n_wide, n_splits, _p(part), _p(tickets), t, self._wait_flag(), 1 if self.use_tcgen05_attention else 0, _DT[q.dtype],
+                self._s()), "attention with mixed heads")
 
     def _tc_attention_takes(self, lib, heads, kv_heads, head_dim, page_size, window, stride) -> bool:
         key = (heads, kv_heads, head_dim, page_size, window, stride)

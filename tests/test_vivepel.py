@@ -307,7 +307,8 @@ def test_one_is_added_to_the_denominator(backend, cuts):
                 w[p + n].mul_(0.1)                      # the biases decide: every query meets every key alike
                 w[p + n + ".b"].zero_()
                 w[p + n + ".b"][10::16] = 4.0 * (sign if n == "q" else 1.0)
-        outs[name] = _mixer_alone(backend, m, cuts, width=32, tweak=tweak)[1]
+        # (scores of -16: the low outputs are e^-16 of a value, and the error of the exponent shows in all of their digits)
+        outs[name] = _mixer_alone(backend, m, cuts, width=32, tweak=tweak, loose=1.0 if name == "high" else 8.0)[1]
     assert float(outs["low"].abs().max()) < 0.02 * float(outs["high"].abs().max())
     assert float(outs["high"][0, 10]) > 3.5             # (the value of the first key as projected, not the normalised key)
 
@@ -366,15 +367,17 @@ def test_runs_of_tokens_in_a_bounded_scratch_buffer(backend, monkeypatch):
 
 
 @pytest.mark.parametrize("backend", CUDA)
-@pytest.mark.parametrize("heads,kv,dim,chunk", [(8, 2, 64, 100), (32, 8, 128, 0), (5, 1, 48, 64), (40, 2, 16, 130)])
-def test_a_batch_of_unequal_requests_is_each_alone(backend, heads, kv, dim, chunk):
+@pytest.mark.parametrize("heads,kv,dim,chunk,ps", [
+    (8, 2, 64, 100, 32), (32, 8, 128, 0, 32), (5, 1, 48, 64, 32), (40, 2, 16, 130, 32), (16, 4, 128, 65, 16), (6, 2, 64, 0, 256), (4, 4, 64, 64, 8),
+    (12, 1, 128, 150, 64), (34, 2, 64, 90, 128)])
+def test_a_batch_of_unequal_requests_is_each_alone(backend, heads, kv, dim, chunk, ps):
     """The kernels themselves on a batch of decoded tokens, short and long portions (some shapes take the prompts' kernels, some the
     decoding ones), against the stand-in; and the same rows for every request whatever stands beside it."""
     from serve_b200.engine.step import BatchShape
     from tests.emu_kernels import EmuKernels
 
     rt, dev = runtime_for(backend)
-    ps, q_lens, lens = 32, [1, 90, 3, 1, 17, 2, 1], [200, 140, 64, 33, 17, 129, 1]
+    q_lens, lens = [1, 290, 3, 1, 17, 2, 1, 70], [200, 340, 64, 33, 17, 129, 1, 70]
     g = torch.Generator().manual_seed(3)
     pages = [-(-n // ps) for n in lens]
     order = torch.randperm(sum(pages), generator=g).tolist()
@@ -385,6 +388,9 @@ def test_a_batch_of_unequal_requests_is_each_alone(backend, heads, kv, dim, chun
             table[r, b] = order.pop()
     rnd = lambda *s: torch.randn(*s, generator=g).to(rt.act_dtype)
     kc, vc = rnd(sum(pages), kv, ps, dim), rnd(sum(pages), kv, ps, dim)
+    for r, n in enumerate(lens):                 # what lies in a page behind a sequence's end is no number
+        kc[table[r, pages[r] - 1], :, n - (pages[r] - 1) * ps:] = float("nan")
+        vc[table[r, pages[r] - 1], :, n - (pages[r] - 1) * ps:] = float("nan")
     q = rnd(sum(q_lens), heads * dim)
     talk = (torch.eye(heads) + 0.3 * torch.randn(heads, heads, generator=g)).to(rt.act_dtype)
     if rt.act_dtype == torch.bfloat16:
@@ -413,6 +419,7 @@ def test_a_batch_of_unequal_requests_is_each_alone(backend, heads, kv, dim, chun
     every = run(list(range(len(lens))), rt.kernels, dev)
     want = run(list(range(len(lens))), EmuKernels("cpu", torch.float64), "cpu")
     torch.testing.assert_close(every, want, atol=_tol(backend, want), rtol=0)
+    rt.kernels.check_errors()
     alone = torch.cat([run([r], rt.kernels, dev) for r in range(len(lens))])
     torch.testing.assert_close(every, alone, atol=_tol(backend, want), rtol=0)
 
