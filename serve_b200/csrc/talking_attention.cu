@@ -332,10 +332,10 @@ __device__ __forceinline__ void token_softmax(const Params& p, int t, int n_tile
   __syncthreads();
 }
 
-// grid (tokens, tile blocks), 4 warps; a warp takes tiles of 64 keys, two strips of 32 at a time. The product is talk [16 MT x Hp]
+// grid (tokens, tile blocks), 4 warps; a warp takes tiles of 64 keys, S strips of 32 at a time. The product is talk [16 MT x Hp]
 // times p [Hp x 32 keys]; column n of the q-th of a strip's four product tiles stands for key 4 n + q, so a lane reads 16 bytes of a
 // head's row and writes 16.
-template <int MT>
+template <int MT, int S>
 __global__ void __launch_bounds__(128) mix_kernel(const Params p) {
   extern __shared__ float mix_s[];
   float *M_s = mix_s, *inv_s = mix_s + p.H;
@@ -358,29 +358,31 @@ __global__ void __launch_bounds__(128) mix_kernel(const Params p) {
       }
       continue;
     }
-    for (int mg = 0; mg < kt_n; mg += MT) {
-      float acc[2][MT][4][4];
+    for (int job = 0; job < (2 / S) * ((kt_n + MT - 1) / MT); ++job) {
+      const int mg = job / (2 / S) * MT, strip0 = job % (2 / S);
+      float acc[S][MT][4][4];
 #pragma unroll
-      for (int s = 0; s < 2; ++s)
+      for (int s = 0; s < S; ++s)
 #pragma unroll
         for (int m = 0; m < MT; ++m)
 #pragma unroll
           for (int n = 0; n < 4; ++n) acc[s][m][n][0] = acc[s][m][n][1] = acc[s][m][n][2] = acc[s][m][n][3] = 0.f;
       for (int kk = 0; kk < kt_n; ++kk) {
-        // heads kk * 16 + 2 tq + {0, 1, 8, 9}: e of four keys each, of both strips
-        float4 ev[2][4];
+        // heads kk * 16 + 2 tq + {0, 1, 8, 9}: e of four keys each, of every strip
+        float4 ev[S][4];
         float f[4];
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
           const int h = kk * 16 + 2 * tq + (i & 1) + ((i >> 1) << 3);
-          const float* src = p.e + (row0 + h) * p.pitch + tile * BN + g * 4;
-          ev[0][i] = h < p.H ? __ldcs(reinterpret_cast<const float4*>(src)) : make_float4(0.f, 0.f, 0.f, 0.f);
-          ev[1][i] = h < p.H ? __ldcs(reinterpret_cast<const float4*>(src + 32)) : make_float4(0.f, 0.f, 0.f, 0.f);
+          const float* src = p.e + (row0 + h) * p.pitch + tile * BN + strip0 * 32 + g * 4;
+#pragma unroll
+          for (int s = 0; s < S; ++s)
+            ev[s][i] = h < p.H ? __ldcs(reinterpret_cast<const float4*>(src + s * 32)) : make_float4(0.f, 0.f, 0.f, 0.f);
           f[i] = h < p.H ? inv_s[h] : 0.f;
           if (!p.fixed && h < p.H) f[i] *= ex2(p.stats[(row0 + h) * tiles_pitch + tile].x - M_s[h]);
         }
 #pragma unroll
-        for (int s = 0; s < 2; ++s) {
+        for (int s = 0; s < S; ++s) {
           uint32_t hi[4][2], lo[4][2];
 #pragma unroll
           for (int j = 0; j < 2; ++j) {
@@ -409,7 +411,7 @@ __global__ void __launch_bounds__(128) mix_kernel(const Params p) {
         }
       }
 #pragma unroll
-      for (int s = 0; s < 2; ++s)
+      for (int s = 0; s < S; ++s)
 #pragma unroll
         for (int m = 0; m < MT; ++m)
 #pragma unroll
@@ -421,7 +423,7 @@ __global__ void __launch_bounds__(128) mix_kernel(const Params p) {
               v.y = pack_bf16(acc[s][m][2][2 * half], acc[s][m][3][2 * half]);
               v.z = pack_bf16(acc[s][m][0][2 * half + 1], acc[s][m][1][2 * half + 1]);
               v.w = pack_bf16(acc[s][m][2][2 * half + 1], acc[s][m][3][2 * half + 1]);
-              *reinterpret_cast<uint4*>((bf16*)p.w + (row0 + h) * p.pitch + tile * BN + s * 32 + tq * 8) = v;
+              *reinterpret_cast<uint4*>((bf16*)p.w + (row0 + h) * p.pitch + tile * BN + (strip0 + s) * 32 + tq * 8) = v;
             }
           }
     }
@@ -526,20 +528,22 @@ __global__ void __launch_bounds__(NW * 32) values_wide_kernel(const Params p) {
   pdl_launch_dependents();
 }
 
-// Requests of at most 16 rows: grid (kv heads, key splits, requests), 4 warps that deal the tiles of the block's keys out among
-// themselves; the warps' sums meet in shared memory, the splits' in the block that arrives last.
+// Requests of at most 16 rows: grid (kv heads, key splits, requests), 4 warps. A block takes 128 keys at a time, a warp 32 of them: a
+// lane looks up where one key lies, and all of the warp's rows are on their way before the first is waited for. The warps' sums meet
+// in shared memory, the splits' in the block that arrives last.
 __global__ void __launch_bounds__(128) values_deep_kernel(const Params p) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   __shared__ int s_last;
+  constexpr int WK = 32;
   pdl_wait();
   const int r = blockIdx.z, hk = blockIdx.x, split = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, tq = lane & 3;
   const int q0 = p.cu_q[r], qn = p.cu_q[r + 1] - q0, M = qn * p.per;
   if (M <= 0 || M > 16 || q0 + qn <= p.t_lo || q0 >= p.t_hi) return;
   const int p0 = p.kv_len[r] - qn;
-  const int lo = first_key(p, p0), hi = p0 + qn, kt0 = lo & ~(BN - 1), n_tiles = (hi - kt0 + BN - 1) / BN;
+  const int lo = first_key(p, p0), hi = p0 + qn, kt0 = lo & ~(BN - 1);
   const int* bt = p.block_table + (size_t)r * p.bt_width;
-  bf16* V = reinterpret_cast<bf16*>(smem_raw) + warp * BN * LDS;
-  const bf16* ws = (const bf16*)p.w;
+  bf16* V = reinterpret_cast<bf16*>(smem_raw) + warp * WK * LDS;
+  const bf16 *ws = (const bf16*)p.w, *vc = (const bf16*)p.vc;
   size_t row[2];
   int pos[2], base[2];
 #pragma unroll
@@ -553,17 +557,23 @@ __global__ void __launch_bounds__(128) values_deep_kernel(const Params p) {
   float o[D / 8][4];
 #pragma unroll
   for (int i = 0; i < D / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-  for (int tile = split * 4 + warp; tile < n_tiles; tile += p.n_splits * 4) {
-    const int kt = kt0 + tile * BN;
-    load_tile<false>(p, (const bf16*)p.vc, bt, hk, kt, lo, hi, V, lane, 32);
+  for (int kt = kt0 + split * 4 * WK + warp * WK; kt < hi; kt += p.n_splits * 4 * WK) {
+    const int key = kt + lane;
+    const long long mine = (key >= lo && key < hi) ? cache_row(p, bt, hk, key) : -1;
+#pragma unroll
+    for (int idx0 = 0; idx0 < WK * CHUNKS; idx0 += 32) {
+      const int idx = idx0 + lane, vrow = idx / CHUNKS, ch = idx - vrow * CHUNKS;
+      const long long off = __shfl_sync(0xffffffffu, mine, vrow);
+      cp_async16(V + vrow * LDS + ch * 8, vc + (off >= 0 ? off + ch * 8 : 0), off >= 0);
+    }
     cp_async_commit();
-    uint32_t wf[BN / 16][4];
+    uint32_t wf[WK / 16][4];
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
-      const bool ok = pos[half] >= 0 && kt >= base[half] && kt <= pos[half];
+      const bool ok = pos[half] >= 0 && kt >= base[half] && (kt & ~(BN - 1)) <= pos[half];
       const bf16* src = ws + row[half] * p.pitch + (kt - base[half]) + tq * 2;
 #pragma unroll
-      for (int kk = 0; kk < BN / 16; ++kk) {
+      for (int kk = 0; kk < WK / 16; ++kk) {
         wf[kk][half] = ok ? *reinterpret_cast<const uint32_t*>(src + kk * 16) : 0u;
         wf[kk][2 + half] = ok ? *reinterpret_cast<const uint32_t*>(src + kk * 16 + 8) : 0u;
       }
@@ -571,7 +581,7 @@ __global__ void __launch_bounds__(128) values_deep_kernel(const Params p) {
     cp_async_wait<0>();
     __syncwarp();
 #pragma unroll
-    for (int kk = 0; kk < BN / 16; ++kk)
+    for (int kk = 0; kk < WK / 16; ++kk)
 #pragma unroll
       for (int d = 0; d < D / 16; ++d) {
         uint32_t b0, b1, b2, b3;
@@ -800,9 +810,9 @@ SB_EXPORT int sb_talking_attention(const void* q, int q_stride, const void* kc, 
     // few tokens: tiles go to blocks of their own; many: a block walks its token's tiles
     const int want = (4 * sm_count() + n_tok - 1) / n_tok, have = (max_tiles + 3) / 4;
     const dim3 grid(n_tok, (unsigned)max(1, min(want, have)));
-    if (H <= 16) SB_PDL_CHECK(launch_pdl(mix_kernel<1>, grid, dim3(128), mix_smem, stream, p));
-    else if (H <= 32) SB_PDL_CHECK(launch_pdl(mix_kernel<2>, grid, dim3(128), mix_smem, stream, p));
-    else SB_PDL_CHECK(launch_pdl(mix_kernel<4>, grid, dim3(128), mix_smem, stream, p));
+    if (H <= 16) SB_PDL_CHECK(launch_pdl(mix_kernel<1, 2>, grid, dim3(128), mix_smem, stream, p));
+    else if (H <= 32) SB_PDL_CHECK(launch_pdl(mix_kernel<2, 1>, grid, dim3(128), mix_smem, stream, p));
+    else SB_PDL_CHECK(launch_pdl(mix_kernel<4, 1>, grid, dim3(128), mix_smem, stream, p));
   }
   if (tc) {
     if (int rc = tc_values(p, max_q, nz, error, stream)) return rc;
@@ -812,7 +822,7 @@ SB_EXPORT int sb_talking_attention(const void* q, int q_stride, const void* kc, 
     SB_PDL_CHECK(launch_pdl(values_wide_kernel<NW>, wgrid, dim3(NW * 32), smem, stream, p));
   }
   if (deep) {
-    const size_t tiles = (size_t)4 * BN * LDS * sizeof(bf16), sums = (size_t)4 * 16 * (D + 2) * sizeof(float);
+    const size_t tiles = (size_t)4 * 32 * LDS * sizeof(bf16), sums = (size_t)4 * 16 * (D + 2) * sizeof(float);
     const size_t smem = tiles > sums ? tiles : sums;
     if (int rc = allow_smem(values_deep_kernel, smem)) return rc;
     SB_PDL_CHECK(launch_pdl(values_deep_kernel, dim3(G, (unsigned)n_splits, R), dim3(128), smem, stream, p));

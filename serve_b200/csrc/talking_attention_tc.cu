@@ -5,7 +5,7 @@
 // column 0. Operands arrive by TMA (128-byte swizzle): queries as a 4-d box, pages of the caches as 4-d boxes named by the block
 // table, mixed weights as a 4-d box of the scratch buffer. One thread issues tcgen05.mma into tensor memory.
 //
-//   scores  S = Q K^T, 128 x 128 a step, two buffers of tensor memory; grid also over runs of keys, since the tiles of one row
+//   scores  S = Q K^T, 128 x 64 a step, two buffers of tensor memory; grid also over runs of keys, since the tiles of one row
 //           tile are independent. Eight warps turn a buffer into exponentials, a thread a row: tcgen05.ld, scale, cap, mask on the
 //           diagonal, exp2, row sums per tile of 64 keys; through shared memory into the scratch rows, 16 bytes a lane.
 //   values  O += W V, 128 x D x 64 a step; O stays in tensor memory. Four warps store it; before, they clear the rows of the first and
@@ -28,20 +28,19 @@ namespace {
 constexpr int D = SB_HEAD_DIM;
 constexpr int KA = D / 64;            // 128-byte swizzle atoms (64 elements) per operand row
 constexpr int BM = 128;               // rows per CTA
-constexpr int SN = 128;               // keys of a score step
-constexpr int RUN = 4;                // score steps a CTA takes
-constexpr int NS_S = 3, NS_V = 3;     // stages
+constexpr int RUN = 8;                // score steps (of 64 keys) a CTA takes
+constexpr int NS_S = 2, NS_V = 3;     // stages (two CTAs of either kernel share an SM)
 constexpr int BT_CACHE = 512;         // block-table entries kept in shared memory
 constexpr unsigned WAIT_LIMIT = 1u << 26;
-constexpr int LDE = 68;               // staging row stride (floats): 64 and 16 bytes of padding
-constexpr int Q_BYTES = BM * D * 2, K_BYTES = SN * D * 2, W_BYTES = BM * BN * 2, V_BYTES = BN * D * 2;
+constexpr int LDE = 36;               // staging row stride (floats): 32 and 16 bytes of padding
+constexpr int Q_BYTES = BM * D * 2, K_BYTES = BN * D * 2, W_BYTES = BM * BN * 2, V_BYTES = BN * D * 2;
 constexpr int EPI = 8;                // epilogue warps of the scores
 constexpr int S_TILES = Q_BYTES + NS_S * K_BYTES, S_STAGE = EPI * 32 * LDE * 4;
 constexpr int S_SMEM = S_TILES + S_STAGE + 256 + BT_CACHE * 4;
 constexpr int V_TILES = NS_V * (W_BYTES + V_BYTES);
 constexpr int V_SMEM = V_TILES + 256 + BT_CACHE * 4;
-constexpr uint32_t S_COLS = 256, V_COLS = D;
-static_assert(S_SMEM <= 227 * 1024, "shared memory");
+constexpr uint32_t S_COLS = 2 * BN, V_COLS = D;
+static_assert(S_SMEM <= 113 * 1024 && V_SMEM <= 113 * 1024, "two CTAs an SM");
 
 __device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void mbar_init(uint64_t* bar, unsigned count) {
@@ -106,6 +105,14 @@ __device__ __forceinline__ uint64_t make_desc(uint32_t smem_addr, uint32_t lbo_b
 }
 __host__ __device__ constexpr uint32_t make_idesc(int m, int n, bool b_mn_major) {
   return (1u << 4) | (1u << 7) | (1u << 10) | ((b_mn_major ? 1u : 0u) << 16) | ((uint32_t)(n >> 3) << 17) | ((uint32_t)(m >> 4) << 24);
+}
+
+// tanh by its Taylor series, for |z| <= SERIES_LIMIT (the first term left out is below 2^-24 of z): no special-function unit, whose
+// two calls per score (three with the exponential) bound the scores otherwise.
+constexpr float SERIES_LIMIT = 0.3f;
+__device__ __forceinline__ float tanh_series(float z) {
+  const float y = z * z;
+  return z * fmaf(y, fmaf(y, fmaf(y, fmaf(y, 62.f / 2835.f, -17.f / 315.f), 2.f / 15.f), -1.f / 3.f), 1.f);
 }
 
 // The index-th row tile of a request, counted from its last (those see most keys): tokens [tok0, tok1) of the request, keys
@@ -178,7 +185,7 @@ __device__ __forceinline__ int load_keys(const Params& p, const CUtensorMap* map
 }
 
 // ------------------------------------------------------------------------------------------------------------ scores
-__global__ void __launch_bounds__(64 + EPI * 32, 1) scores_tc_kernel(const __grid_constant__ CUtensorMap map_q,
+__global__ void __launch_bounds__(64 + EPI * 32, 2) scores_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                                                                      const __grid_constant__ CUtensorMap map_k, const Params p, int n_runs,
                                                                      int* error) {
   extern __shared__ __align__(1024) unsigned char smem[];
@@ -192,13 +199,13 @@ __global__ void __launch_bounds__(64 + EPI * 32, 1) scores_tc_kernel(const __gri
   Tile w;
   if (!find_tile(p, blockIdx.y / n_runs, w)) return;
   const int run = blockIdx.y % n_runs;
-  const int n_steps_all = (w.hi - w.kt0 + SN - 1) / SN, step0 = run * RUN, n_steps = min(n_steps_all - step0, RUN);
+  const int n_steps_all = (w.hi - w.kt0 + BN - 1) / BN, step0 = run * RUN, n_steps = min(n_steps_all - step0, RUN);
   if (n_steps <= 0) return;
   if ((smem_u32(smem) & 1023u) != 0) {                        // never seen; refuse rather than compute with a wrong swizzle
     if (threadIdx.x == 0) atomicExch(error, 1);
     return;
   }
-  const int kt_first = w.kt0 + step0 * SN;
+  const int kt_first = w.kt0 + step0 * BN;
   if (threadIdx.x == 0) {
     mbar_init(&q_full, 1);
 #pragma unroll
@@ -220,39 +227,34 @@ __global__ void __launch_bounds__(64 + EPI * 32, 1) scores_tc_kernel(const __gri
 
   if (warp == 0) {
     int bt_first;
-    const int* bt = table_of(p, w, max(kt_first, w.lo), min(kt_first + n_steps * SN, w.hi), bt_s, lane, bt_first);
+    const int* bt = table_of(p, w, max(kt_first, w.lo), min(kt_first + n_steps * BN, w.hi), bt_s, lane, bt_first);
     if (lane == 0) {
       mbar_expect_tx(&q_full, (unsigned)(tpt * p.per * D * 2));
 #pragma unroll
       for (int a = 0; a < KA; ++a) tma_load_4d(Qs + (size_t)a * BM * 128, &map_q, &q_full, a * 64, 0, w.hk, w.q0 + w.tok0);
       const unsigned box = (unsigned)((p.ps < BN ? p.ps : BN) * D * 2);
       for (int j = 0; j < n_steps; ++j) {
-        const int s = j % NS_S, kt = kt_first + j * SN;
+        const int s = j % NS_S, kt = kt_first + j * BN;
         if (!mbar_wait(&k_empty[s], ((j / NS_S) & 1) ^ 1)) { failed = true; break; }
-        unsigned char* dst = Ks + (size_t)s * K_BYTES;
-        int n = 0;
-#pragma unroll
-        for (int half = 0; half < 2; ++half) n += load_keys(p, &map_k, bt, bt_first, w.hk, kt + half * BN, w.lo, w.hi, nullptr, 0, nullptr);
-        mbar_expect_tx(&k_full[s], n * box);
-#pragma unroll
-        for (int half = 0; half < 2; ++half)
-          load_keys(p, &map_k, bt, bt_first, w.hk, kt + half * BN, w.lo, w.hi, dst + half * BN * 128, SN * 128, &k_full[s]);
+        mbar_expect_tx(&k_full[s], load_keys(p, &map_k, bt, bt_first, w.hk, kt, w.lo, w.hi, nullptr, 0, nullptr) * box);
+        load_keys(p, &map_k, bt, bt_first, w.hk, kt, w.lo, w.hi, Ks + (size_t)s * K_BYTES, BN * 128, &k_full[s]);
       }
     }
   } else if (warp == 1) {
     if (lane == 0) {
-      constexpr uint32_t idesc = make_idesc(BM, SN, false);
+      constexpr uint32_t idesc = make_idesc(BM, BN, false);
       const uint64_t dq = make_desc(smem_u32(Qs), 0);
       failed = !mbar_wait(&q_full, 0);
       for (int j = 0; j < n_steps && !failed; ++j) {
         if (!mbar_wait(&k_full[j % NS_S], (j / NS_S) & 1) || !mbar_wait(&s_empty[j & 1], ((j >> 1) & 1) ^ 1)) { failed = true; break; }
         tc_fence_after();
         const uint64_t dk = make_desc(smem_u32(Ks + (size_t)(j % NS_S) * K_BYTES), 0);
-        const uint32_t acc = tmem_base + (uint32_t)((j & 1) * SN);
+        const uint32_t acc = tmem_base + (uint32_t)((j & 1) * BN);
 #pragma unroll
         for (int kk = 0; kk < D / 16; ++kk) {
-          const uint64_t off = (uint64_t)((kk >> 2) * (BM * 128 >> 4) + (kk & 3) * 2);      // (both operands have 128 rows an atom)
-          tc_mma(acc, dq + off, dk + off, idesc, kk != 0 ? 1u : 0u);
+          // 16 k-values further: 32 bytes within an atom (4 steps), then the next atom of Q (128 rows) and K (64 rows)
+          const uint64_t qo = (uint64_t)((kk >> 2) * (BM * 128 >> 4) + (kk & 3) * 2), ko = (uint64_t)((kk >> 2) * (BN * 128 >> 4) + (kk & 3) * 2);
+          tc_mma(acc, dq + qo, dk + ko, idesc, kk != 0 ? 1u : 0u);
         }
         tc_commit(&s_full[j & 1]);
         tc_commit(&k_empty[j % NS_S]);
@@ -265,69 +267,75 @@ __global__ void __launch_bounds__(64 + EPI * 32, 1) scores_tc_kernel(const __gri
     const int pos = row_ok ? w.p0 + w.tok0 + tok : -1;
     const size_t srow = row_ok ? (size_t)(w.q0 + w.tok0 + tok - p.t_lo) * p.H + w.hk * p.per + (row - tok * p.per) : 0;
     float* stage = reinterpret_cast<float*>(smem + S_TILES) + (warp - 2) * 32 * LDE;
-    const uint32_t lane_addr = tmem_base + ((uint32_t)(q * 32) << 16) + (uint32_t)(set * SN);
+    const uint32_t lane_addr = tmem_base + ((uint32_t)(q * 32) << 16) + (uint32_t)(set * BN);
     const int first_pos = w.p0 + w.tok0;                      // smallest position of the tile's rows
     const float two_in = p.cap_in * (2.f * LOG2E), cap_log2 = p.cap * LOG2E, scale_log2 = p.scale * LOG2E;
     const int tiles_pitch = p.pitch / BN;
     for (int j = set; j < n_steps && !failed; j += 2) {
       if (!mbar_wait(&s_full[set], (j >> 1) & 1)) { failed = true; break; }
       tc_fence_after();
-#pragma unroll 1
-      for (int half = 0; half < 2; ++half) {
-        const int kt = kt_first + j * SN + half * BN;
-        float v[BN];
-        tc_load32(lane_addr + (uint32_t)(half * BN), v);
-        tc_load32(lane_addr + (uint32_t)(half * BN + 32), v + 32);
-        tc_wait_ld();
-        if (half == 1) {
-          tc_fence_before();
-          __syncwarp();
-          if (lane == 0) mbar_arrive(&s_empty[set]);          // the scores are in registers: the buffer may be used again
-        }
-        const bool live = kt <= pos;                          // the row reads keys of this tile (its first key is never behind it)
-        if (!__any_sync(0xffffffffu, live)) continue;
-        if (p.cap > 0.f) {
+      const int kt = kt_first + j * BN;
+      float v[BN];
+      tc_load32(lane_addr, v);
+      tc_load32(lane_addr + 32u, v + 32);
+      tc_wait_ld();
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&s_empty[set]);              // the scores are in registers: the buffer may be used again
+      const bool live = kt <= pos;                            // the row reads keys of this tile (its first key is never behind it)
+      if (!__any_sync(0xffffffffu, live)) continue;
+      if (p.cap > 0.f) {
+        float big = 0.f;
 #pragma unroll
-          for (int i = 0; i < BN; ++i) v[i] = capped_log2(v[i], two_in, cap_log2);
+        for (int i = 0; i < BN; ++i) big = fmaxf(big, fabsf(v[i]));
+        if (__all_sync(0xffffffffu, big * p.cap_in <= SERIES_LIMIT)) {
+#pragma unroll
+          for (int i = 0; i < BN; ++i) v[i] = cap_log2 * tanh_series(v[i] * p.cap_in);
         } else {
 #pragma unroll
-          for (int i = 0; i < BN; ++i) v[i] *= scale_log2;
+          for (int i = 0; i < BN; ++i) v[i] = capped_log2(v[i], two_in, cap_log2);
         }
-        if (kt + BN - 1 > first_pos || kt < w.lo) {
+      } else {
 #pragma unroll
-          for (int i = 0; i < BN; ++i) v[i] = (kt + i <= pos && kt + i >= w.lo) ? v[i] : -INFINITY;
-        }
-        float m = 0.f;
-        if (!p.fixed) {
-          m = -INFINITY;
+        for (int i = 0; i < BN; ++i) v[i] *= scale_log2;
+      }
+      if (kt + BN - 1 > first_pos || kt < w.lo) {
 #pragma unroll
-          for (int i = 0; i < BN; ++i) m = fmaxf(m, v[i]);
-        }
+        for (int i = 0; i < BN; ++i) v[i] = (kt + i <= pos && kt + i >= w.lo) ? v[i] : -INFINITY;
+      }
+      float m = 0.f;
+      if (!p.fixed) {
+        m = -INFINITY;
+#pragma unroll
+        for (int i = 0; i < BN; ++i) m = fmaxf(m, v[i]);
         const float ref = (m == -INFINITY) ? 0.f : m;
-        float s0 = 0.f, s1 = 0.f;
 #pragma unroll
-        for (int i = 0; i < BN; i += 4) {
+        for (int i = 0; i < BN; ++i) v[i] -= ref;
+      }
+      float s0 = 0.f, s1 = 0.f;
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+#pragma unroll
+        for (int i = 0; i < 32; i += 4) {
           float4 e;
-          e.x = ex2(v[i] - ref); e.y = ex2(v[i + 1] - ref); e.z = ex2(v[i + 2] - ref); e.w = ex2(v[i + 3] - ref);
+          e.x = ex2(v[half * 32 + i]); e.y = ex2(v[half * 32 + i + 1]); e.z = ex2(v[half * 32 + i + 2]); e.w = ex2(v[half * 32 + i + 3]);
           s0 += e.x + e.y;
           s1 += e.z + e.w;
           *reinterpret_cast<float4*>(stage + lane * LDE + i) = e;
         }
-        if (live) p.stats[srow * tiles_pitch + (kt - w.kt0) / BN] = make_float2(m, s0 + s1);
         __syncwarp();
-        // two rows an instruction: lanes 0-15 one, 16-31 the next, 16 bytes each
-#pragma unroll 4
-        for (int i = 0; i < 32; i += 2) {
-          const int rr = i + (lane >> 4);
-          const int ok = __shfl_sync(0xffffffffu, (int)live, rr);
-          const unsigned lo32 = __shfl_sync(0xffffffffu, (unsigned)srow, rr);
-          if (ok) {
-            float* dst = p.e + (size_t)lo32 * p.pitch + (kt - w.kt0) + (lane & 15) * 4;
-            *reinterpret_cast<float4*>(dst) = *reinterpret_cast<const float4*>(stage + rr * LDE + (lane & 15) * 4);
-          }
+        // four rows an instruction: eight lanes a row, 16 bytes each
+        float* dst0 = p.e + (kt - w.kt0) + half * 32 + (lane & 7) * 4;
+#pragma unroll
+        for (int i = 0; i < 32; i += 4) {
+          const int rr = i + (lane >> 3);
+          const unsigned at = __shfl_sync(0xffffffffu, live ? (unsigned)srow : 0xffffffffu, rr);
+          if (at != 0xffffffffu)
+            *reinterpret_cast<float4*>(dst0 + (size_t)at * p.pitch) = *reinterpret_cast<const float4*>(stage + rr * LDE + (lane & 7) * 4);
         }
         __syncwarp();
       }
+      if (live) p.stats[srow * tiles_pitch + (kt - w.kt0) / BN] = make_float2(m, s0 + s1);
     }
   }
   if (failed) atomicExch(error, 1);
@@ -511,7 +519,7 @@ int tc_scores(const Params& p, int n_tokens, int max_keys, int max_q, int n_requ
   CUtensorMap map_q, map_k;
   if (int rc = encode_rows(&map_q, p.q, p, n_tokens, D, p.q_stride)) return rc;
   if (int rc = encode_cache(&map_k, p.kc, p)) return rc;
-  const int n_runs = ((max_keys + SN - 1) / SN + RUN - 1) / RUN;
+  const int n_runs = ((max_keys + BN - 1) / BN + RUN - 1) / RUN;
   const long long y = (long long)row_tiles(p, max_q) * n_runs;
   if (y > 65535) return SB_ERR_LIMIT;
   cudaFuncSetAttribute(scores_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, S_SMEM);

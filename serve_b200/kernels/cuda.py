@@ -799,7 +799,7 @@ class CudaKernels:
         step = max(1, min(t, self.TALK_SCRATCH_BYTES // per_token))
         n_splits, part, tickets = 1, None, None
         if bf16 and which & 2:
-            n_splits = max(1, min(-(-2 * self.TARGET_BLOCKS // (shape.rows * kv_heads)), -(-pitch // 256), self.MAX_SPLITS))
+            n_splits = max(1, min(-(-4 * self.TARGET_BLOCKS // (shape.rows * kv_heads)), -(-pitch // 128), self.MAX_SPLITS))
             if n_splits > 1:
                 part = torch.empty((shape.rows, kv_heads, n_splits, 16, head_dim), dtype=torch.float32, device=q.device)
                 tickets = self._ticket_buffer(shape.rows * kv_heads)
