@@ -409,12 +409,12 @@ def gebilorn_at(width: int, vocab: int = 32000):
 
 def vivepel_at(width: int, vocab: int = 32000):
     """A Vivepel configuration with layers of a real model's sizes: attention with mixed heads of 128 (half of a head rotated, blocks
-    of 1,024 positions, capped scores) and a dense feed-forward with as many weights as the Llama decoder's gated one; norms over
+    of 1,536 positions, capped scores) and a dense feed-forward with as many weights as the Llama decoder's gated one; norms over
     eight parts of the row."""
     from serve_b200.config import config_from_dict
 
     heads, _experts, top, ff = DESIGN_SIZES[str(width)]
-    att = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 0.08, "softcap": 30.0, "mask": {"size": 1024},
+    att = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 0.08, "softcap": 30.0, "mask": {"size": 1536},
            "rot": {"base": 500000.0, "dims": 64}}
     layers = [{"type": "attention", "mixer": att, "mlp": {"kind": "dense", "ff": 3 * top * ff // 2}}] * 3
     return config_from_dict({"architecture": "Vivepel", "width": width, "vocab": vocab, "norm": {"eps": 1e-5, "groups": 8}, "layers": layers,

@@ -31,26 +31,25 @@ __device__ __forceinline__ void store4(bf16* p, float4 v) {
 __device__ __forceinline__ float dot4(float4 v) { return (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w); }
 __device__ __forceinline__ float4 mul4(float4 v, float f, float4 w) { return make_float4(v.x * f * w.x, v.y * f * w.y, v.z * f * w.z, v.w * f * w.w); }
 
-// A block's sum; a block of one warp needs no shared memory.
-__device__ __forceinline__ float team_sum(float v, float* red) { return blockDim.x <= 32 ? warp_sum(v) : block_sum(v, red); }
-
 struct NormArgs {
   float* x; const void* delta; const float* through; const int* rows; const float* weight; void* out;
   int dim, part; float eps;        // row length, length of a part
 };
 
-// grid (rows, groups). The part stays in registers: VPT float4 a thread. x null: out = the norm of delta.
-template <typename TD, typename TO, int VPT>
-__global__ void __launch_bounds__(512) grouped_norm_vec_kernel(const NormArgs a) {
-  __shared__ float red[32];
-  const int src = a.rows ? a.rows[blockIdx.x] : (int)blockIdx.x;
-  const int off = blockIdx.y * a.part, nvec = a.part >> 2;
-  const TD* dr = a.delta ? (const TD*)a.delta + (size_t)src * a.dim + off : nullptr;
-  float* xr = a.x ? a.x + (size_t)src * a.dim + off : nullptr;
+// The part stays in registers: VPT float4 a thread of its team, a block (grid: row, part), or, WARP, a warp (short parts: the
+// blocks deal the parts of all rows out to their warps). x null: out = the norm of delta.
+template <typename TD, typename TO, int VPT, bool WARP>
+__global__ void __launch_bounds__(512) grouped_norm_vec_kernel(const NormArgs a, int n_parts, int groups) {
+  __shared__ float red[WARP ? 1 : 32];
+  const int team = WARP ? blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5) : (int)blockIdx.x;
+  if (team >= n_parts) { pdl_wait(); return; }                // (a whole team; a block's only team never leaves)
+  const int at = WARP ? threadIdx.x & 31 : threadIdx.x, step = WARP ? 32 : blockDim.x;
+  const int r = team / groups, off = (team - r * groups) * a.part, nvec = a.part >> 2;
+  auto sum = [&](float v) { return WARP ? warp_sum(v) : block_sum(v, red); };
   float4 d[VPT], v[VPT], w[VPT], wd[VPT];
 #pragma unroll
   for (int k = 0; k < VPT; ++k) {        // weights: no kernel of a step writes them
-    const int i = threadIdx.x + k * blockDim.x;
+    const int i = at + k * step;
     w[k] = wd[k] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (i < nvec) {
       w[k] = load4(a.weight + off + i * 4);
@@ -59,10 +58,13 @@ __global__ void __launch_bounds__(512) grouped_norm_vec_kernel(const NormArgs a)
   }
   pdl_launch_dependents();
   pdl_wait();
+  const int src = a.rows ? a.rows[r] : r;
+  const TD* dr = a.delta ? (const TD*)a.delta + (size_t)src * a.dim + off : nullptr;
+  float* xr = a.x ? a.x + (size_t)src * a.dim + off : nullptr;
   float ss = 0.f;
 #pragma unroll
   for (int k = 0; k < VPT; ++k) {
-    const int i = threadIdx.x + k * blockDim.x;
+    const int i = at + k * step;
     d[k] = v[k] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (i < nvec) {
       if (dr) d[k] = load4(dr + i * 4);
@@ -71,7 +73,7 @@ __global__ void __launch_bounds__(512) grouped_norm_vec_kernel(const NormArgs a)
     ss += dot4(d[k]);
   }
   if (a.through) {
-    const float inv = 1.0f / sqrtf(team_sum(ss, red) / (float)a.part + a.eps);
+    const float inv = 1.0f / sqrtf(sum(ss) / (float)a.part + a.eps);
 #pragma unroll
     for (int k = 0; k < VPT; ++k) d[k] = mul4(d[k], inv, wd[k]);
   }
@@ -81,11 +83,11 @@ __global__ void __launch_bounds__(512) grouped_norm_vec_kernel(const NormArgs a)
     v[k].x += d[k].x; v[k].y += d[k].y; v[k].z += d[k].z; v[k].w += d[k].w;
     ss += dot4(v[k]);
   }
-  const float inv = 1.0f / sqrtf(team_sum(ss, red) / (float)a.part + a.eps);
-  TO* orow = (TO*)a.out + (size_t)blockIdx.x * a.dim + off;
+  const float inv = 1.0f / sqrtf(sum(ss) / (float)a.part + a.eps);
+  TO* orow = (TO*)a.out + (size_t)r * a.dim + off;
 #pragma unroll
   for (int k = 0; k < VPT; ++k) {
-    const int i = threadIdx.x + k * blockDim.x;
+    const int i = at + k * step;
     if (i < nvec) {
       if (xr && dr && !a.rows) store4(xr + i * 4, v[k]);
       store4(orow + i * 4, mul4(v[k], inv, w[k]));
@@ -130,22 +132,32 @@ __global__ void __launch_bounds__(256) grouped_norm_kernel(const NormArgs a) {
 
 template <typename TD, typename TO>
 int launch_grouped_norm(const NormArgs& a, int n_rows, int groups, cudaStream_t stream) {
-  const dim3 grid(n_rows, groups);
   const int nvec = a.part / 4;
   if (a.part % 4 == 0 && nvec <= 512 * 4 && (!a.x || aligned16(a.x)) && (!a.delta || aligned16(a.delta)) && (!a.through || aligned16(a.through)) &&
       aligned16(a.weight) && aligned16(a.out)) {
-    const int threads = nvec <= 32 ? 32 : (nvec <= 64 ? 64 : (nvec <= 128 ? 128 : (nvec <= 512 ? 256 : 512)));
+    const int n_parts = n_rows * groups;
+#define SB_GROUPED(VPT, WARP, BLOCKS, THREADS)                                                                                         \
+  SB_PDL_CHECK(launch_pdl(grouped_norm_vec_kernel<TD, TO, VPT, WARP>, dim3(BLOCKS), dim3(THREADS), 0, stream, a, n_parts, groups))
+    if (nvec <= 128) {
+      const int warps = n_parts >= 4 * sm_count() ? 8 : 1, blocks = (n_parts + warps - 1) / warps;
+      if (nvec <= 32) SB_GROUPED(1, true, blocks, warps * 32);
+      else if (nvec <= 64) SB_GROUPED(2, true, blocks, warps * 32);
+      else SB_GROUPED(4, true, blocks, warps * 32);
+      return 0;
+    }
+    const int threads = nvec <= 512 ? 256 : 512;
     const int vpt = (nvec + threads - 1) / threads;
-    if (vpt <= 1) SB_PDL_CHECK(launch_pdl(grouped_norm_vec_kernel<TD, TO, 1>, grid, dim3(threads), 0, stream, a));
-    else if (vpt <= 2) SB_PDL_CHECK(launch_pdl(grouped_norm_vec_kernel<TD, TO, 2>, grid, dim3(threads), 0, stream, a));
-    else SB_PDL_CHECK(launch_pdl(grouped_norm_vec_kernel<TD, TO, 4>, grid, dim3(threads), 0, stream, a));
+    if (vpt <= 1) SB_GROUPED(1, false, n_parts, threads);
+    else if (vpt <= 2) SB_GROUPED(2, false, n_parts, threads);
+    else SB_GROUPED(4, false, n_parts, threads);
+#undef SB_GROUPED
     return 0;
   }
   const size_t smem = (size_t)a.part * sizeof(float);
   if (smem > 200 * 1024) return SB_ERR_LIMIT;
   auto k = grouped_norm_kernel<TD, TO>;
   if (smem > 40 * 1024) cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-  k<<<grid, a.part <= 64 ? 64 : 256, smem, stream>>>(a);
+  k<<<dim3(n_rows, groups), a.part <= 64 ? 64 : 256, smem, stream>>>(a);
   SB_LAUNCH_CHECK();
   return 0;
 }

@@ -6,6 +6,7 @@
 //                             with the logarithm of the position; keys and values into their cache pages
 //   sb_latent_prepare         latent attention: the latent vector normalised, the shared key part and every head's
 //                             rotated query part turned by position; one cache row per token
+//   sb_qk_prepare             float sums of a query | key | value projection: bias, norm, partial rotation, cache write
 //   sb_gated_activation       act(gate, up) of a fused gate/up product: silu(g) * u, the clamped form
 //                             g <- min(g, limit), u <- clamp(u, -limit, limit), g * sigmoid(alpha g) * (u + 1), or
 //                             gelu(g) * u with the tanh form of gelu
@@ -394,9 +395,9 @@ __global__ void __launch_bounds__(256) add_bias_kernel(float* __restrict__ x, co
 // by the angle position * inv_freq[i]; queries to q_out [T, H * D], keys and values to their page. Everything is float
 // until the one rounding at the store. The row (with its bias) and the token's cosines and sines are kept in shared
 // memory, so the sums are read from memory once (rows of up to 200 KB). With head_norm every query and key head is
-// instead divided, after its rotation, by its own root mean square over its dim true elements, without a weight; with
-// head_norm 2 before its rotation, and multiplied by a weight [D] that all query (all key) heads share. With keys_are_values
-// the row ends with the keys, [T, (H + G) * D], and the value pages take the keys as projected, before norm and rotation.
+// instead divided, after its rotation, by its own root mean square over its dim true elements, without a weight. With
+// keys_are_values the row ends with the keys, [T, (H + G) * D], and the value pages take the keys as projected, before norm and
+// rotation.
 template <typename T>
 __global__ void __launch_bounds__(512) qk_prepare_kernel(
     const float* __restrict__ sums, int stride, const float* __restrict__ bias, const int* __restrict__ positions,
@@ -409,7 +410,6 @@ __global__ void __launch_bounds__(512) qk_prepare_kernel(
   const float* row = sums + (size_t)t * stride;
   const int nq = H * D, nk = G * D, half = rot >> 1;
   const int n_all = nq + (keys_are_values ? 1 : 2) * nk;
-  const bool whole_norm = head_norm == 0;
   float* cs_table = dyn;
   float* vals = dyn + (rot > 0 ? rot : 2);
   const int pos = positions[t];
@@ -424,8 +424,8 @@ __global__ void __launch_bounds__(512) qk_prepare_kernel(
     else if (i < nq + nk) sk += v * v;
   }
   float inv_q = 1.f, inv_k = 1.f;
-  if (q_weight != nullptr && whole_norm) inv_q = 1.0f / sqrtf(block_sum(sq, red) / (float)(H * dim) + eps);
-  if (k_weight != nullptr && whole_norm && G > 0) inv_k = 1.0f / sqrtf(block_sum(sk, red) / (float)(G * dim) + eps);
+  if (q_weight != nullptr) inv_q = 1.0f / sqrtf(block_sum(sq, red) / (float)(H * dim) + eps);
+  if (k_weight != nullptr && G > 0) inv_k = 1.0f / sqrtf(block_sum(sk, red) / (float)(G * dim) + eps);
   __syncthreads();                          // the table and the row are whole
   // A warp takes a head at a time, a lane an element; an element below rot / 2 is turned together with its partner rot / 2
   // further on, so every value is normalised once. Heads 0 .. H-1 are queries, the G after them keys.
@@ -439,14 +439,10 @@ __global__ void __launch_bounds__(512) qk_prepare_kernel(
     const bool is_q = head < H;
     if (!is_q && !page_ok) continue;
     const float* w = is_q ? q_weight : k_weight;
-    float inv = is_q ? inv_q : inv_k;
-    const int base = head * D, w_base = head_norm == 2 ? 0 : (is_q ? base : base - nq);
+    const float inv = is_q ? inv_q : inv_k;
+    const int base = head * D, w_base = is_q ? base : base - nq;
     T* dst = is_q ? q_out + (size_t)t * q_stride + base : kc + (((size_t)page * G + (head - H)) * ps + within) * D;
-    if (head_norm == 2) {
-      float ss = 0.f;
-      for (int d = lane; d < D; d += 32) ss += vals[base + d] * vals[base + d];      // (zero beyond the head's true size)
-      inv = 1.0f / sqrtf(warp_sum(ss) / (float)dim + eps);
-    } else if (head_norm) {
+    if (head_norm) {
       // the head is turned in place in shared memory (a lane turns an element together with its partner), its squares are
       // summed over the warp, and the quotient is stored
       float ss = 0.f;
@@ -489,6 +485,89 @@ __global__ void __launch_bounds__(512) qk_prepare_kernel(
   for (int i = threadIdx.x; i < nk; i += blockDim.x) {
     const int g = i / D, d = i - g * D;
     vc[(((size_t)page * G + g) * ps + within) * D + d] = from_float<T>(values[i]);
+  }
+}
+
+// The same preparation where every query and key head has a norm of its own before the rotation, with a weight [D] that all query (all
+// key) heads share: heads stand alone, so a warp takes one at a time, four elements a lane, and a block the heads of one token, whose
+// cosines and sines it keeps. Float until the one rounding at the store.
+template <typename T>
+__global__ void __launch_bounds__(512) head_norm_prepare_kernel(
+    const float* __restrict__ sums, int stride, const float* __restrict__ bias, const int* __restrict__ positions,
+    const int* __restrict__ token_row, int H, int G, int D, int dim, const float* __restrict__ q_weight, const float* __restrict__ k_weight,
+    float eps, const float* __restrict__ inv_freq, int rot, T* __restrict__ q_out, int q_stride, T* __restrict__ kc, T* __restrict__ vc,
+    const int* __restrict__ block_table, int bt_width, int ps, int num_pages, int* __restrict__ errors, int keys_are_values) {
+  extern __shared__ __align__(16) float dyn[];         // [half] cosines, [half] sines, then a row of D floats a warp
+  const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
+  const int half = rot >> 1, n_heads = H + G + (keys_are_values ? 0 : G), D4 = D >> 2;
+  float *cs = dyn, *sn = dyn + half, *row = dyn + ((rot + 3) & ~3) + warp * D;
+  const float* src = sums + (size_t)t * stride;
+  pdl_wait();
+  auto fetch = [&](int head, float4 (&v)[2]) {
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+      const int i = lane + 32 * k;
+      v[k] = i < D4 ? reinterpret_cast<const float4*>(src + (size_t)head * D)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+  };
+  float4 v[2], ahead[2];
+  if (warp < n_heads) fetch(warp, ahead);
+  const int pos = positions[t], blk = ps > 0 ? pos / ps : 0;
+  const int page = (G > 0 && pos >= 0 && blk < bt_width) ? block_table[(size_t)token_row[t] * bt_width + blk] : -1;
+  const bool page_ok = page >= 0 && page < num_pages;
+  if (G > 0 && !page_ok && threadIdx.x == 0) atomicAdd(errors, 1);
+  for (int j = threadIdx.x; j < half; j += blockDim.x) sincosf((float)pos * inv_freq[j], &sn[j], &cs[j]);
+  __syncthreads();
+  for (int head = warp; head < n_heads; head += n_warps) {
+    v[0] = ahead[0];
+    v[1] = ahead[1];
+    if (head + n_warps < n_heads) fetch(head + n_warps, ahead);
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+      const int i = lane + 32 * k;
+      if (i < D4 && bias) {
+        const float4 b = reinterpret_cast<const float4*>(bias + (size_t)head * D)[i];
+        v[k].x += b.x; v[k].y += b.y; v[k].z += b.z; v[k].w += b.w;
+      }
+      ss += (v[k].x * v[k].x + v[k].y * v[k].y) + (v[k].z * v[k].z + v[k].w * v[k].w);      // (zero beyond the head's true size)
+    }
+    const bool is_q = head < H, is_k = !is_q && head < H + G;
+    const size_t cell = is_q ? 0 : (((size_t)page * G + (head - H) % G) * ps + (pos - blk * ps)) * D;
+    if (!is_q && !page_ok) continue;
+    if (!is_q && (keys_are_values || !is_k)) {
+#pragma unroll
+      for (int k = 0; k < 2; ++k)
+        if (lane + 32 * k < D4) store4f<T>(vc + cell + (lane + 32 * k) * 4, v[k]);
+      if (!is_k) continue;
+    }
+    const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)dim + eps);
+    const float* w = is_q ? q_weight : k_weight;
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+      const int i = lane + 32 * k;
+      if (i < D4) {
+        const float4 u = reinterpret_cast<const float4*>(w)[i];
+        v[k].x *= inv * u.x; v[k].y *= inv * u.y; v[k].z *= inv * u.z; v[k].w *= inv * u.w;
+        if (i * 4 < rot) reinterpret_cast<float4*>(row)[i] = v[k];
+      }
+    }
+    __syncwarp();
+    T* dst = is_q ? q_out + (size_t)t * q_stride + (size_t)head * D : kc + cell;
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+      const int i = lane + 32 * k;
+      if (i >= D4) continue;
+      float e[4] = {v[k].x, v[k].y, v[k].z, v[k].w};
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        const int d = i * 4 + c;
+        if (d < half) e[c] = e[c] * cs[d] - row[d + half] * sn[d];
+        else if (d < rot) e[c] = e[c] * cs[d - half] + row[d - half] * sn[d - half];
+      }
+      store4f<T>(dst + i * 4, make_float4(e[0], e[1], e[2], e[3]));
+    }
+    __syncwarp();
   }
 }
 
@@ -562,6 +641,26 @@ SB_EXPORT int sb_qk_prepare(const float* sums, int stride, const float* bias, co
   if (H <= 0 || G < 0 || D <= 0 || dim <= 0 || dim > D || stride < n_all || head_norm < 0 || head_norm > 2 || (head_norm == 2 && (!q_weight || (G > 0 && !k_weight))) || q_stride < H * D) return SB_ERR_SHAPE;
   if (rot < 0 || (rot & 1) || rot > dim || (rot > 0 && !inv_freq)) return SB_ERR_SHAPE;
   if (G > 0 && (ps <= 0 || bt_width <= 0 || !kc || !vc || !errors)) return SB_ERR_SHAPE;
+  if (head_norm == 2) {
+    if (D % 4 || D > 256 || stride % 4 || q_stride % 4 || !aligned16(sums) || (bias && !aligned16(bias)) || !aligned16(q_weight) ||
+        (G > 0 && (!aligned16(k_weight) || !aligned16(kc) || !aligned16(vc))) || !aligned16(q_out))
+      return SB_ERR_ALIGN;
+    // few tokens: as many warps as a token has heads, so that each takes one or two
+    const int heads = n_all / D, warps = n_tokens >= 4 * sm_count() ? 8 : (heads < 16 ? heads : 16);
+    const size_t bytes = ((size_t)((rot + 3) & ~3) + (size_t)warps * D) * sizeof(float);
+    if (bytes > 48 * 1024) return SB_ERR_LIMIT;
+    if (dtype == SB_DTYPE_F32)
+      SB_PDL_CHECK(launch_pdl(head_norm_prepare_kernel<float>, dim3(n_tokens), dim3(warps * 32), bytes, stream, sums, stride, bias, positions,
+                              token_row, H, G, D, dim, q_weight, k_weight, eps, inv_freq, rot, (float*)q_out, q_stride, (float*)kc, (float*)vc,
+                              block_table, bt_width, ps, num_pages, errors, keys_are_values));
+    else if (dtype == SB_DTYPE_BF16)
+      SB_PDL_CHECK(launch_pdl(head_norm_prepare_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(warps * 32), bytes, stream, sums, stride, bias,
+                              positions, token_row, H, G, D, dim, q_weight, k_weight, eps, inv_freq, rot, (__nv_bfloat16*)q_out, q_stride,
+                              (__nv_bfloat16*)kc, (__nv_bfloat16*)vc, block_table, bt_width, ps, num_pages, errors, keys_are_values));
+    else
+      return SB_ERR_DTYPE;
+    return 0;
+  }
   const size_t smem = ((size_t)(rot > 0 ? rot : 2) + (size_t)n_all) * sizeof(float);
   if (smem > 200 * 1024) return SB_ERR_LIMIT;
   const int threads = n_all >= 2048 ? 512 : 256;

@@ -332,10 +332,10 @@ __device__ __forceinline__ void token_softmax(const Params& p, int t, int n_tile
   __syncthreads();
 }
 
-// grid (tokens, tile blocks), 4 warps; a warp takes tiles of 64 keys, S strips of 32 at a time. The product is talk [16 MT x Hp]
-// times p [Hp x 32 keys]; column n of the q-th of a strip's four product tiles stands for key 4 n + q, so a lane reads 16 bytes of a
-// head's row and writes 16.
-template <int MT, int S>
+// grid (tokens, tile blocks), 4 warps; a warp takes tiles of 64 keys, a strip of 32 at a time. The product is talk [16 MT x Hp] times
+// p [Hp x 32 keys], 16 heads g a step; column n of the q-th of a strip's four product tiles stands for key 4 n + q, so a lane reads 16
+// bytes of a head's row and writes 16. A step's rows are fetched while the step before it is computed.
+template <int MT>
 __global__ void __launch_bounds__(128) mix_kernel(const Params p) {
   extern __shared__ float mix_s[];
   float *M_s = mix_s, *inv_s = mix_s + p.H;
@@ -345,89 +345,98 @@ __global__ void __launch_bounds__(128) mix_kernel(const Params p) {
   const int base = first_key(p, pos) & ~(BN - 1), n_tiles = (pos - base) / BN + 1;
   const int n_all = p.zero_ahead ? min((pos + p.zero_ahead - base) / BN + 1, p.pitch / BN) : n_tiles;
   if ((int)blockIdx.y * 4 >= n_all) return;
-  const int tiles_pitch = p.pitch / BN;
-  token_softmax(p, t, n_tiles, M_s, inv_s);
+  const int tiles_pitch = p.pitch / BN, tile_step = gridDim.y * 4;
   const int kt_n = (p.H + 15) / 16, hp = kt_n * 16;
   const uint32_t* talk = reinterpret_cast<const uint32_t*>(p.talk);     // pairs of neighbouring columns
   const size_t row0 = (size_t)t * p.H;
-  for (int tile = blockIdx.y * 4 + warp; tile < n_all; tile += gridDim.y * 4) {
-    if (tile >= n_tiles) {
-      for (int h = g; h < p.H; h += 8) {
-        uint4* dst = reinterpret_cast<uint4*>((bf16*)p.w + (row0 + h) * p.pitch + tile * BN + tq * 16);
-        dst[0] = dst[1] = make_uint4(0, 0, 0, 0);
-      }
-      continue;
+  // heads kk * 16 + 2 tq + {0, 1, 8, 9}: e of four keys each
+  auto head_of = [&](int kk, int i) { return kk * 16 + 2 * tq + (i & 1) + ((i >> 1) << 3); };
+  auto fetch = [&](int tile, int strip, int kk, float4 (&ev)[4]) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int h = head_of(kk, i);
+      ev[i] = h < p.H ? __ldcs(reinterpret_cast<const float4*>(p.e + (row0 + h) * p.pitch + tile * BN + strip * 32 + g * 4))
+                      : make_float4(0.f, 0.f, 0.f, 0.f);
     }
-    for (int job = 0; job < (2 / S) * ((kt_n + MT - 1) / MT); ++job) {
-      const int mg = job / (2 / S) * MT, strip0 = job % (2 / S);
-      float acc[S][MT][4][4];
+  };
+  int tile = blockIdx.y * 4 + warp, strip = 0, mg = 0, kk = 0;
+  float4 next[4];
+  if (tile < n_tiles) fetch(tile, 0, 0, next);
+  token_softmax(p, t, n_tiles, M_s, inv_s);
+  float acc[MT][4][4];
+  while (tile < n_tiles) {
+    float4 ev[4];
 #pragma unroll
-      for (int s = 0; s < S; ++s)
+    for (int i = 0; i < 4; ++i) ev[i] = next[i];
+    const int at_tile = tile, at_strip = strip, at_mg = mg, at_kk = kk;
+    if (++kk == kt_n) {
+      kk = 0;
+      mg += MT;
+      if (mg >= kt_n) {
+        mg = 0;
+        strip ^= 1;
+        if (strip == 0) tile += tile_step;
+      }
+    }
+    if (tile < n_tiles) fetch(tile, strip, kk, next);
+    if (at_kk == 0) {
 #pragma unroll
-        for (int m = 0; m < MT; ++m)
+      for (int m = 0; m < MT; ++m)
 #pragma unroll
-          for (int n = 0; n < 4; ++n) acc[s][m][n][0] = acc[s][m][n][1] = acc[s][m][n][2] = acc[s][m][n][3] = 0.f;
-      for (int kk = 0; kk < kt_n; ++kk) {
-        // heads kk * 16 + 2 tq + {0, 1, 8, 9}: e of four keys each, of every strip
-        float4 ev[S][4];
-        float f[4];
+        for (int n = 0; n < 4; ++n) acc[m][n][0] = acc[m][n][1] = acc[m][n][2] = acc[m][n][3] = 0.f;
+    }
+    uint32_t hi[4][2], lo[4][2];
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const int h = kk * 16 + 2 * tq + (i & 1) + ((i >> 1) << 3);
-          const float* src = p.e + (row0 + h) * p.pitch + tile * BN + strip0 * 32 + g * 4;
+    for (int j = 0; j < 2; ++j) {
+      float f[2];
 #pragma unroll
-          for (int s = 0; s < S; ++s)
-            ev[s][i] = h < p.H ? __ldcs(reinterpret_cast<const float4*>(src + s * 32)) : make_float4(0.f, 0.f, 0.f, 0.f);
-          f[i] = h < p.H ? inv_s[h] : 0.f;
-          if (!p.fixed && h < p.H) f[i] *= ex2(p.stats[(row0 + h) * tiles_pitch + tile].x - M_s[h]);
-        }
+      for (int i = 0; i < 2; ++i) {
+        const int h = head_of(at_kk, 2 * j + i);
+        f[i] = h < p.H ? inv_s[h] : 0.f;
+        if (!p.fixed && h < p.H) f[i] *= ex2(p.stats[(row0 + h) * tiles_pitch + at_tile].x - M_s[h]);
+      }
+      const float4 a = ev[2 * j], b = ev[2 * j + 1];
+      const float xs[4] = {a.x * f[0], a.y * f[0], a.z * f[0], a.w * f[0]}, ys[4] = {b.x * f[1], b.y * f[1], b.z * f[1], b.w * f[1]};
 #pragma unroll
-        for (int s = 0; s < S; ++s) {
-          uint32_t hi[4][2], lo[4][2];
+      for (int n = 0; n < 4; ++n) {
+        const __nv_bfloat162 h2 = __floats2bfloat162_rn(xs[n], ys[n]);
+        hi[n][j] = *reinterpret_cast<const uint32_t*>(&h2);
+        lo[n][j] = pack_bf16(xs[n] - __low2float(h2), ys[n] - __high2float(h2));
+      }
+    }
 #pragma unroll
-          for (int j = 0; j < 2; ++j) {
-            const float4 a = ev[s][2 * j], b = ev[s][2 * j + 1];
-            const float fa = f[2 * j], fb = f[2 * j + 1];
-            const float xs[4] = {a.x * fa, a.y * fa, a.z * fa, a.w * fa}, ys[4] = {b.x * fb, b.y * fb, b.z * fb, b.w * fb};
+    for (int m = 0; m < MT; ++m) {
+      if (at_mg + m < kt_n) {
+        const uint32_t* a = talk + ((size_t)((at_mg + m) * 16 + g) * hp + at_kk * 16) / 2 + tq;
+        const uint32_t a0 = __ldg(a), a1 = __ldg(a + 4 * hp), a2 = __ldg(a + 4), a3 = __ldg(a + 4 * hp + 4);
 #pragma unroll
-            for (int n = 0; n < 4; ++n) {
-              const __nv_bfloat162 h2 = __floats2bfloat162_rn(xs[n], ys[n]);
-              hi[n][j] = *reinterpret_cast<const uint32_t*>(&h2);
-              lo[n][j] = pack_bf16(xs[n] - __low2float(h2), ys[n] - __high2float(h2));
-            }
-          }
-#pragma unroll
-          for (int m = 0; m < MT; ++m) {
-            if (mg + m < kt_n) {
-              const uint32_t* a = talk + ((size_t)((mg + m) * 16 + g) * hp + kk * 16) / 2 + tq;
-              const uint32_t a0 = __ldg(a), a1 = __ldg(a + 4 * hp), a2 = __ldg(a + 4), a3 = __ldg(a + 4 * hp + 4);
-#pragma unroll
-              for (int n = 0; n < 4; ++n) {
-                mma_bf16(acc[s][m][n], a0, a1, a2, a3, lo[n][0], lo[n][1]);
-                mma_bf16(acc[s][m][n], a0, a1, a2, a3, hi[n][0], hi[n][1]);
-              }
-            }
-          }
+        for (int n = 0; n < 4; ++n) {
+          mma_bf16(acc[m][n], a0, a1, a2, a3, lo[n][0], lo[n][1]);
+          mma_bf16(acc[m][n], a0, a1, a2, a3, hi[n][0], hi[n][1]);
         }
       }
-#pragma unroll
-      for (int s = 0; s < S; ++s)
-#pragma unroll
-        for (int m = 0; m < MT; ++m)
-#pragma unroll
-          for (int half = 0; half < 2; ++half) {
-            const int h = (mg + m) * 16 + g + 8 * half;
-            if (h < p.H) {
-              uint4 v;
-              v.x = pack_bf16(acc[s][m][0][2 * half], acc[s][m][1][2 * half]);
-              v.y = pack_bf16(acc[s][m][2][2 * half], acc[s][m][3][2 * half]);
-              v.z = pack_bf16(acc[s][m][0][2 * half + 1], acc[s][m][1][2 * half + 1]);
-              v.w = pack_bf16(acc[s][m][2][2 * half + 1], acc[s][m][3][2 * half + 1]);
-              *reinterpret_cast<uint4*>((bf16*)p.w + (row0 + h) * p.pitch + tile * BN + (strip0 + s) * 32 + tq * 8) = v;
-            }
-          }
     }
+    if (at_kk != kt_n - 1) continue;
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int h = (at_mg + m) * 16 + g + 8 * half;
+        if (h < p.H) {
+          uint4 v;
+          v.x = pack_bf16(acc[m][0][2 * half], acc[m][1][2 * half]);
+          v.y = pack_bf16(acc[m][2][2 * half], acc[m][3][2 * half]);
+          v.z = pack_bf16(acc[m][0][2 * half + 1], acc[m][1][2 * half + 1]);
+          v.w = pack_bf16(acc[m][2][2 * half + 1], acc[m][3][2 * half + 1]);
+          *reinterpret_cast<uint4*>((bf16*)p.w + (row0 + h) * p.pitch + at_tile * BN + at_strip * 32 + tq * 8) = v;
+        }
+      }
   }
+  for (; tile < n_all; tile += tile_step)
+    for (int h = g; h < p.H; h += 8) {
+      uint4* dst = reinterpret_cast<uint4*>((bf16*)p.w + (row0 + h) * p.pitch + tile * BN + tq * 16);
+      dst[0] = dst[1] = make_uint4(0, 0, 0, 0);
+    }
 }
 
 // float32: a block per (token, tile of 64 keys); the tile's weights of all heads in shared memory (in parts of 128 heads).
@@ -810,9 +819,9 @@ SB_EXPORT int sb_talking_attention(const void* q, int q_stride, const void* kc, 
     // few tokens: tiles go to blocks of their own; many: a block walks its token's tiles
     const int want = (4 * sm_count() + n_tok - 1) / n_tok, have = (max_tiles + 3) / 4;
     const dim3 grid(n_tok, (unsigned)max(1, min(want, have)));
-    if (H <= 16) SB_PDL_CHECK(launch_pdl(mix_kernel<1, 2>, grid, dim3(128), mix_smem, stream, p));
-    else if (H <= 32) SB_PDL_CHECK(launch_pdl(mix_kernel<2, 1>, grid, dim3(128), mix_smem, stream, p));
-    else SB_PDL_CHECK(launch_pdl(mix_kernel<4, 1>, grid, dim3(128), mix_smem, stream, p));
+    if (H <= 16) SB_PDL_CHECK(launch_pdl(mix_kernel<1>, grid, dim3(128), mix_smem, stream, p));
+    else if (H <= 32) SB_PDL_CHECK(launch_pdl(mix_kernel<2>, grid, dim3(128), mix_smem, stream, p));
+    else SB_PDL_CHECK(launch_pdl(mix_kernel<4>, grid, dim3(128), mix_smem, stream, p));
   }
   if (tc) {
     if (int rc = tc_values(p, max_q, nz, error, stream)) return rc;

@@ -28,7 +28,7 @@ namespace {
 constexpr int D = SB_HEAD_DIM;
 constexpr int KA = D / 64;            // 128-byte swizzle atoms (64 elements) per operand row
 constexpr int BM = 128;               // rows per CTA
-constexpr int RUN = 8;                // score steps (of 64 keys) a CTA takes
+constexpr int RUN = 16;               // score steps (of 64 keys) a CTA takes: 4 to 24 measured, a CTA's start costs about three steps
 constexpr int NS_S = 2, NS_V = 3;     // stages (two CTAs of either kernel share an SM)
 constexpr int BT_CACHE = 512;         // block-table entries kept in shared memory
 constexpr unsigned WAIT_LIMIT = 1u << 26;

@@ -769,7 +769,7 @@ class CudaKernels:
             ctypes.c_float(softcap), _p(sinks), kv_div, keep_first, self._s()), "attention")
 
     # Scratch bytes a launch of the mixed-head attention may use; a step that needs more runs in runs of tokens.
-    TALK_SCRATCH_BYTES = int(os.environ.get("SERVE_B200_TALK_SCRATCH", str(512 << 20)))
+    TALK_SCRATCH_BYTES = int(os.environ.get("SERVE_B200_TALK_SCRATCH", str(1 << 30)))
 
     def talking_attention(self, q, k_cache, v_cache, block_table, cu_q, kv_len, positions, heads, kv_heads, head_dim, page_size, scale,
                           talk, out, shape, chunk: int = 0, softcap: float = 0.0, sinks=None) -> None:
