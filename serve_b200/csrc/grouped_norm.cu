@@ -271,7 +271,9 @@ SB_EXPORT int sb_poly_norm(const void* z, const float* coef, float eps, void* ou
   if (dtype == SB_DTYPE_BF16) {
     const int nvec = n / 8;
     if (n % 8 == 0 && nvec <= 512 * 8 && aligned16(z) && aligned16(out)) {
-      const int threads = nvec <= 32 ? 32 : (nvec <= 128 ? 64 : (nvec <= 512 ? 256 : 512));
+      // many rows: small blocks with much in flight; few: as many threads as there is work for
+      const bool many = n_rows >= 4 * sm_count();
+      const int threads = nvec <= 32 ? 32 : (nvec <= 128 ? 64 : (many && nvec <= 1024 ? 128 : (nvec <= 512 || (many && nvec <= 2048) ? 256 : 512)));
       const int vpt = (nvec + threads - 1) / threads;
       if (vpt <= 2) SB_PDL_CHECK(launch_pdl(poly_norm_vec_kernel<2>, dim3(n_rows), dim3(threads), 0, stream, (const bf16*)z, coef, eps, (bf16*)out, n));
       else if (vpt <= 4) SB_PDL_CHECK(launch_pdl(poly_norm_vec_kernel<4>, dim3(n_rows), dim3(threads), 0, stream, (const bf16*)z, coef, eps, (bf16*)out, n));

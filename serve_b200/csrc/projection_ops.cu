@@ -491,26 +491,28 @@ __global__ void __launch_bounds__(512) qk_prepare_kernel(
 // The same preparation where every query and key head has a norm of its own before the rotation, with a weight [D] that all query (all
 // key) heads share: heads stand alone, so a warp takes one at a time, four elements a lane, and a block the heads of one token, whose
 // cosines and sines it keeps. Float until the one rounding at the store.
-template <typename T>
+// KV: float4 a lane (D <= 128 KV).
+template <typename T, int KV>
 __global__ void __launch_bounds__(512) head_norm_prepare_kernel(
     const float* __restrict__ sums, int stride, const float* __restrict__ bias, const int* __restrict__ positions,
     const int* __restrict__ token_row, int H, int G, int D, int dim, const float* __restrict__ q_weight, const float* __restrict__ k_weight,
     float eps, const float* __restrict__ inv_freq, int rot, T* __restrict__ q_out, int q_stride, T* __restrict__ kc, T* __restrict__ vc,
     const int* __restrict__ block_table, int bt_width, int ps, int num_pages, int* __restrict__ errors, int keys_are_values) {
-  extern __shared__ __align__(16) float dyn[];         // [half] cosines, [half] sines, then a row of D floats a warp
+  extern __shared__ __align__(16) float dyn[];         // cosines, sines (each padded to a multiple of 4), then a row of D floats a warp
   const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
   const int half = rot >> 1, n_heads = H + G + (keys_are_values ? 0 : G), D4 = D >> 2;
-  float *cs = dyn, *sn = dyn + half, *row = dyn + ((rot + 3) & ~3) + warp * D;
+  const int half4 = (half + 3) & ~3;
+  float *cs = dyn, *sn = dyn + half4, *row = dyn + 2 * half4 + warp * D;
   const float* src = sums + (size_t)t * stride;
   pdl_wait();
-  auto fetch = [&](int head, float4 (&v)[2]) {
+  auto fetch = [&](int head, float4 (&v)[KV]) {
 #pragma unroll
-    for (int k = 0; k < 2; ++k) {
+    for (int k = 0; k < KV; ++k) {
       const int i = lane + 32 * k;
       v[k] = i < D4 ? reinterpret_cast<const float4*>(src + (size_t)head * D)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
     }
   };
-  float4 v[2], ahead[2];
+  float4 ahead[KV];
   if (warp < n_heads) fetch(warp, ahead);
   const int pos = positions[t], blk = ps > 0 ? pos / ps : 0;
   const int page = (G > 0 && pos >= 0 && blk < bt_width) ? block_table[(size_t)token_row[t] * bt_width + blk] : -1;
@@ -519,12 +521,13 @@ __global__ void __launch_bounds__(512) head_norm_prepare_kernel(
   for (int j = threadIdx.x; j < half; j += blockDim.x) sincosf((float)pos * inv_freq[j], &sn[j], &cs[j]);
   __syncthreads();
   for (int head = warp; head < n_heads; head += n_warps) {
-    v[0] = ahead[0];
-    v[1] = ahead[1];
+    float4 v[KV];
+#pragma unroll
+    for (int k = 0; k < KV; ++k) v[k] = ahead[k];
     if (head + n_warps < n_heads) fetch(head + n_warps, ahead);
     float ss = 0.f;
 #pragma unroll
-    for (int k = 0; k < 2; ++k) {
+    for (int k = 0; k < KV; ++k) {
       const int i = lane + 32 * k;
       if (i < D4 && bias) {
         const float4 b = reinterpret_cast<const float4*>(bias + (size_t)head * D)[i];
@@ -533,18 +536,18 @@ __global__ void __launch_bounds__(512) head_norm_prepare_kernel(
       ss += (v[k].x * v[k].x + v[k].y * v[k].y) + (v[k].z * v[k].z + v[k].w * v[k].w);      // (zero beyond the head's true size)
     }
     const bool is_q = head < H, is_k = !is_q && head < H + G;
-    const size_t cell = is_q ? 0 : (((size_t)page * G + (head - H) % G) * ps + (pos - blk * ps)) * D;
+    const size_t cell = is_q ? 0 : (((size_t)page * G + (head < H + G ? head - H : head - H - G)) * ps + (pos - blk * ps)) * D;
     if (!is_q && !page_ok) continue;
     if (!is_q && (keys_are_values || !is_k)) {
 #pragma unroll
-      for (int k = 0; k < 2; ++k)
+      for (int k = 0; k < KV; ++k)
         if (lane + 32 * k < D4) store4f<T>(vc + cell + (lane + 32 * k) * 4, v[k]);
       if (!is_k) continue;
     }
     const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)dim + eps);
     const float* w = is_q ? q_weight : k_weight;
 #pragma unroll
-    for (int k = 0; k < 2; ++k) {
+    for (int k = 0; k < KV; ++k) {
       const int i = lane + 32 * k;
       if (i < D4) {
         const float4 u = reinterpret_cast<const float4*>(w)[i];
@@ -555,9 +558,22 @@ __global__ void __launch_bounds__(512) head_norm_prepare_kernel(
     __syncwarp();
     T* dst = is_q ? q_out + (size_t)t * q_stride + (size_t)head * D : kc + cell;
 #pragma unroll
-    for (int k = 0; k < 2; ++k) {
+    for (int k = 0; k < KV; ++k) {
       const int i = lane + 32 * k;
       if (i >= D4) continue;
+      if (i * 4 >= rot) {
+        store4f<T>(dst + i * 4, v[k]);
+        continue;
+      }
+      if ((half & 3) == 0) {                          // a lane's four partners are neighbours too
+        const int q4 = half >> 2, at = i < q4 ? i : i - q4;
+        const float4 o = reinterpret_cast<const float4*>(row)[i < q4 ? i + q4 : at];
+        const float4 c = reinterpret_cast<const float4*>(cs)[at];
+        float4 s = reinterpret_cast<const float4*>(sn)[at];
+        if (i < q4) { s.x = -s.x; s.y = -s.y; s.z = -s.z; s.w = -s.w; }
+        store4f<T>(dst + i * 4, make_float4(v[k].x * c.x + o.x * s.x, v[k].y * c.y + o.y * s.y, v[k].z * c.z + o.z * s.z, v[k].w * c.w + o.w * s.w));
+        continue;
+      }
       float e[4] = {v[k].x, v[k].y, v[k].z, v[k].w};
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
@@ -645,20 +661,18 @@ SB_EXPORT int sb_qk_prepare(const float* sums, int stride, const float* bias, co
     if (D % 4 || D > 256 || stride % 4 || q_stride % 4 || !aligned16(sums) || (bias && !aligned16(bias)) || !aligned16(q_weight) ||
         (G > 0 && (!aligned16(k_weight) || !aligned16(kc) || !aligned16(vc))) || !aligned16(q_out))
       return SB_ERR_ALIGN;
-    // few tokens: as many warps as a token has heads, so that each takes one or two
-    const int heads = n_all / D, warps = n_tokens >= 4 * sm_count() ? 8 : (heads < 16 ? heads : 16);
-    const size_t bytes = ((size_t)((rot + 3) & ~3) + (size_t)warps * D) * sizeof(float);
+    // few tokens: as many warps as a token has heads, so that each takes one or two; many: small blocks, whose starts overlap
+    const int heads = n_all / D, warps = n_tokens >= 4 * sm_count() ? 4 : (heads < 16 ? heads : 16);
+    const size_t bytes = ((size_t)2 * ((rot / 2 + 3) & ~3) + (size_t)warps * D) * sizeof(float);
     if (bytes > 48 * 1024) return SB_ERR_LIMIT;
-    if (dtype == SB_DTYPE_F32)
-      SB_PDL_CHECK(launch_pdl(head_norm_prepare_kernel<float>, dim3(n_tokens), dim3(warps * 32), bytes, stream, sums, stride, bias, positions,
-                              token_row, H, G, D, dim, q_weight, k_weight, eps, inv_freq, rot, (float*)q_out, q_stride, (float*)kc, (float*)vc,
-                              block_table, bt_width, ps, num_pages, errors, keys_are_values));
-    else if (dtype == SB_DTYPE_BF16)
-      SB_PDL_CHECK(launch_pdl(head_norm_prepare_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(warps * 32), bytes, stream, sums, stride, bias,
-                              positions, token_row, H, G, D, dim, q_weight, k_weight, eps, inv_freq, rot, (__nv_bfloat16*)q_out, q_stride,
-                              (__nv_bfloat16*)kc, (__nv_bfloat16*)vc, block_table, bt_width, ps, num_pages, errors, keys_are_values));
-    else
-      return SB_ERR_DTYPE;
+#define SB_HEAD_NORM(T, KV)                                                                                                                 \
+  SB_PDL_CHECK(launch_pdl(head_norm_prepare_kernel<T, KV>, dim3(n_tokens), dim3(warps * 32), bytes, stream, sums, stride, bias, positions,    \
+                          token_row, H, G, D, dim, q_weight, k_weight, eps, inv_freq, rot, (T*)q_out, q_stride, (T*)kc, (T*)vc, block_table, \
+                          bt_width, ps, num_pages, errors, keys_are_values))
+    if (dtype == SB_DTYPE_F32) { if (D <= 128) SB_HEAD_NORM(float, 1); else SB_HEAD_NORM(float, 2); }
+    else if (dtype == SB_DTYPE_BF16) { if (D <= 128) SB_HEAD_NORM(__nv_bfloat16, 1); else SB_HEAD_NORM(__nv_bfloat16, 2); }
+    else return SB_ERR_DTYPE;
+#undef SB_HEAD_NORM
     return 0;
   }
   const size_t smem = ((size_t)(rot > 0 ? rot : 2) + (size_t)n_all) * sizeof(float);

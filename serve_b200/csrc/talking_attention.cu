@@ -10,6 +10,8 @@
 //   mix     per token: the tiles' (m, sum) give every head's maximum and denominator; p = e * exp(m - M) / den, mixed over the heads
 //   values  per (request, kv head, rows): the product of mixed weights and values
 //
+// (a step of few rows mixes inside the values' kernel: two passes)
+//
 // Scratch rows: token t (counted from the first token of the launch), head h, ``pitch`` keys, column 0 standing for the key
 // base(t) = the first key the token may read, rounded down to a tile of 64. Tiles never depend on how a prompt was cut or on
 // what else is in the batch. A query sees the keys j <= i, with ``chunk`` > 0 only those of its own block of chunk positions.
@@ -34,6 +36,9 @@ constexpr int D = SB_HEAD_DIM;
 constexpr int LDS = D + 8;           // row stride of a key or value tile in shared memory (elements)
 constexpr int LDW = BN + 8;          // row stride of a weight tile in shared memory
 constexpr int CHUNKS = D / 8;        // 16-byte pieces per row
+// shared memory of the deep values: four warps' 32 value rows, over which their sums [4][16][D + 2] lie afterwards
+constexpr size_t DEEP_TILES = (size_t)4 * 32 * LDS * 2, DEEP_SUMS = (size_t)4 * 16 * (D + 2) * 4;
+constexpr size_t DEEP_BYTES = ((DEEP_TILES > DEEP_SUMS ? DEEP_TILES : DEEP_SUMS) + 15) / 16 * 16;
 static_assert(D % 16 == 0 && D >= 16 && D <= 256, "head_dim must be a multiple of 16 in 16..256");
 
 __device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -539,7 +544,10 @@ __global__ void __launch_bounds__(NW * 32) values_wide_kernel(const Params p) {
 
 // Requests of at most 16 rows: grid (kv heads, key splits, requests), 4 warps. A block takes 128 keys at a time, a warp 32 of them: a
 // lane looks up where one key lies, and all of the warp's rows are on their way before the first is waited for. The warps' sums meet
-// in shared memory, the splits' in the block that arrives last.
+// in shared memory, the splits' in the block that arrives last. FUSED: the step has few rows and no wide request, and the block mixes the weights
+// itself, for the heads of its kv head only (every kv head's blocks read all heads' exponentials; a step of few rows has few of
+// them), so no mixed weights are written and read.
+template <bool FUSED>
 __global__ void __launch_bounds__(128) values_deep_kernel(const Params p) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   __shared__ int s_last;
@@ -563,28 +571,100 @@ __global__ void __launch_bounds__(128) values_deep_kernel(const Params p) {
     row[half] = ok ? (size_t)(t - p.t_lo) * p.H + hk * p.per + (m - tok * p.per) : 0;
     base[half] = ok ? first_key(p, pos[half]) & ~(BN - 1) : 0;
   }
-  float o[D / 8][4];
-#pragma unroll
-  for (int i = 0; i < D / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-  for (int kt = kt0 + split * 4 * WK + warp * WK; kt < hi; kt += p.n_splits * 4 * WK) {
+  // FUSED: a strip's keys come out of the mix in the order 4 n + q (product tile q, column n): the value rows are laid out likewise
+  auto fetch = [&](int kt) {
     const int key = kt + lane;
     const long long mine = (key >= lo && key < hi) ? cache_row(p, bt, hk, key) : -1;
 #pragma unroll
     for (int idx0 = 0; idx0 < WK * CHUNKS; idx0 += 32) {
       const int idx = idx0 + lane, vrow = idx / CHUNKS, ch = idx - vrow * CHUNKS;
       const long long off = __shfl_sync(0xffffffffu, mine, vrow);
-      cp_async16(V + vrow * LDS + ch * 8, vc + (off >= 0 ? off + ch * 8 : 0), off >= 0);
+      const int at = FUSED ? ((vrow & 3) << 3) + (vrow >> 2) : vrow;
+      cp_async16(V + at * LDS + ch * 8, vc + (off >= 0 ? off + ch * 8 : 0), off >= 0);
     }
     cp_async_commit();
-    uint32_t wf[WK / 16][4];
+  };
+  const int step = p.n_splits * 4 * WK;
+  int kt = kt0 + (split * 4 + warp) * WK;
+  if (kt < hi) fetch(kt);
+  float *M_s = reinterpret_cast<float*>(smem_raw + DEEP_BYTES), *inv_s = M_s + 16 * p.G;      // [token][H]
+  if (FUSED) {
+    for (int i = 0; i < qn; ++i) {
+      const int t = q0 + i;
+      if (t < p.t_lo || t >= p.t_hi) continue;
+      token_softmax(p, t - p.t_lo, (p0 + i - (first_key(p, p0 + i) & ~(BN - 1))) / BN + 1, M_s + i * p.H, inv_s + i * p.H);
+    }
+  }
+  float o[D / 8][4];
 #pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      const bool ok = pos[half] >= 0 && kt >= base[half] && (kt & ~(BN - 1)) <= pos[half];
-      const bf16* src = ws + row[half] * p.pitch + (kt - base[half]) + tq * 2;
+  for (int i = 0; i < D / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+  for (bool fetched = true; kt < hi; kt += step, fetched = false) {
+    if (!fetched) fetch(kt);
+    uint32_t wf[WK / 16][4];
+    if (FUSED) {
+      float acc[4][4];
+#pragma unroll
+      for (int n = 0; n < 4; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
+      const int kt_n = (p.H + 15) / 16, hp = kt_n * 16;
+      const uint32_t* talk = reinterpret_cast<const uint32_t*>(p.talk);
+      const int m_a = g, m_b = g + 8, tok_a = m_a / p.per, tok_b = m_b / p.per;
+      for (int i = 0; i < qn; ++i) {
+        // this token's rows of the product's first operand, the others' are zero: the sum over the tokens holds every row
+        const int t = q0 + i, at_pos = p0 + i, at_base = first_key(p, at_pos) & ~(BN - 1);
+        if (t < p.t_lo || t >= p.t_hi || kt < at_base || (kt & ~(BN - 1)) > at_pos) continue;
+        const size_t row0 = (size_t)(t - p.t_lo) * p.H;
+        const bool use_a = m_a < M && tok_a == i, use_b = m_b < M && tok_b == i;
+        const uint32_t* ta = talk + (size_t)(use_a ? hk * p.per + (m_a - tok_a * p.per) : 0) * (hp / 2) + tq;
+        const uint32_t* tb = talk + (size_t)(use_b ? hk * p.per + (m_b - tok_b * p.per) : 0) * (hp / 2) + tq;
+        for (int kk = 0; kk < kt_n; ++kk) {
+          float4 ev[4];
+          float f[4];
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            const int h = kk * 16 + 2 * tq + (j & 1) + ((j >> 1) << 3);
+            ev[j] = h < p.H ? *reinterpret_cast<const float4*>(p.e + (row0 + h) * p.pitch + (kt - at_base) + g * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+            f[j] = h < p.H ? inv_s[i * p.H + h] : 0.f;
+            if (!p.fixed && h < p.H) f[j] *= ex2(p.stats[(row0 + h) * (p.pitch / BN) + (kt - at_base) / BN].x - M_s[i * p.H + h]);
+          }
+          const uint32_t a0 = use_a ? __ldg(ta + kk * 8) : 0u, a2 = use_a ? __ldg(ta + kk * 8 + 4) : 0u;
+          const uint32_t a1 = use_b ? __ldg(tb + kk * 8) : 0u, a3 = use_b ? __ldg(tb + kk * 8 + 4) : 0u;
+          uint32_t hi2[4][2], lo2[4][2];
+#pragma unroll
+          for (int j = 0; j < 2; ++j) {
+            const float4 a = ev[2 * j], b = ev[2 * j + 1];
+            const float xs[4] = {a.x * f[2 * j], a.y * f[2 * j], a.z * f[2 * j], a.w * f[2 * j]};
+            const float ys[4] = {b.x * f[2 * j + 1], b.y * f[2 * j + 1], b.z * f[2 * j + 1], b.w * f[2 * j + 1]};
+#pragma unroll
+            for (int n = 0; n < 4; ++n) {
+              const __nv_bfloat162 h2 = __floats2bfloat162_rn(xs[n], ys[n]);
+              hi2[n][j] = *reinterpret_cast<const uint32_t*>(&h2);
+              lo2[n][j] = pack_bf16(xs[n] - __low2float(h2), ys[n] - __high2float(h2));
+            }
+          }
+#pragma unroll
+          for (int n = 0; n < 4; ++n) {
+            mma_bf16(acc[n], a0, a1, a2, a3, lo2[n][0], lo2[n][1]);
+            mma_bf16(acc[n], a0, a1, a2, a3, hi2[n][0], hi2[n][1]);
+          }
+        }
+      }
 #pragma unroll
       for (int kk = 0; kk < WK / 16; ++kk) {
-        wf[kk][half] = ok ? *reinterpret_cast<const uint32_t*>(src + kk * 16) : 0u;
-        wf[kk][2 + half] = ok ? *reinterpret_cast<const uint32_t*>(src + kk * 16 + 8) : 0u;
+        wf[kk][0] = pack_bf16(acc[2 * kk][0], acc[2 * kk][1]);
+        wf[kk][1] = pack_bf16(acc[2 * kk][2], acc[2 * kk][3]);
+        wf[kk][2] = pack_bf16(acc[2 * kk + 1][0], acc[2 * kk + 1][1]);
+        wf[kk][3] = pack_bf16(acc[2 * kk + 1][2], acc[2 * kk + 1][3]);
+      }
+    } else {
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const bool ok = pos[half] >= 0 && kt >= base[half] && (kt & ~(BN - 1)) <= pos[half];
+        const bf16* src = ws + row[half] * p.pitch + (kt - base[half]) + tq * 2;
+#pragma unroll
+        for (int kk = 0; kk < WK / 16; ++kk) {
+          wf[kk][half] = ok ? *reinterpret_cast<const uint32_t*>(src + kk * 16) : 0u;
+          wf[kk][2 + half] = ok ? *reinterpret_cast<const uint32_t*>(src + kk * 16 + 8) : 0u;
+        }
       }
     }
     cp_async_wait<0>();
@@ -815,7 +895,9 @@ SB_EXPORT int sb_talking_attention(const void* q, int q_stride, const void* kc, 
     SB_PDL_CHECK(launch_pdl(scores_wide_kernel<NW>, wgrid, dim3(NW * 32), smem, stream, p));
   }
   if (deep) SB_PDL_CHECK(launch_pdl(scores_deep_kernel, dim3(G, (unsigned)((max_tiles + 3) / 4), R), dim3(128), 0, stream, p));
-  {
+  // (with more (request, kv head) pairs than SMs, every pair mixing for itself costs more than the launch it saves)
+  const bool fused = !wide && R * G <= sm_count();
+  if (!fused) {
     // few tokens: tiles go to blocks of their own; many: a block walks its token's tiles
     const int want = (4 * sm_count() + n_tok - 1) / n_tok, have = (max_tiles + 3) / 4;
     const dim3 grid(n_tok, (unsigned)max(1, min(want, have)));
@@ -831,10 +913,16 @@ SB_EXPORT int sb_talking_attention(const void* q, int q_stride, const void* kc, 
     SB_PDL_CHECK(launch_pdl(values_wide_kernel<NW>, wgrid, dim3(NW * 32), smem, stream, p));
   }
   if (deep) {
-    const size_t tiles = (size_t)4 * 32 * LDS * sizeof(bf16), sums = (size_t)4 * 16 * (D + 2) * sizeof(float);
-    const size_t smem = tiles > sums ? tiles : sums;
-    if (int rc = allow_smem(values_deep_kernel, smem)) return rc;
-    SB_PDL_CHECK(launch_pdl(values_deep_kernel, dim3(G, (unsigned)n_splits, R), dim3(128), smem, stream, p));
+    const size_t smem = DEEP_BYTES + (!fused ? 0 : (size_t)2 * 16 * G * sizeof(float));      // (a request's tokens times H: at most 16 G)
+    if (smem > 200 * 1024) return SB_ERR_LIMIT;
+    const dim3 grid(G, (unsigned)n_splits, R);
+    if (!fused) {
+      if (int rc = allow_smem(values_deep_kernel<false>, smem)) return rc;
+      SB_PDL_CHECK(launch_pdl(values_deep_kernel<false>, grid, dim3(128), smem, stream, p));
+    } else {
+      if (int rc = allow_smem(values_deep_kernel<true>, smem)) return rc;
+      SB_PDL_CHECK(launch_pdl(values_deep_kernel<true>, grid, dim3(128), smem, stream, p));
+    }
   }
   return 0;
 }

@@ -28,7 +28,8 @@ namespace {
 constexpr int D = SB_HEAD_DIM;
 constexpr int KA = D / 64;            // 128-byte swizzle atoms (64 elements) per operand row
 constexpr int BM = 128;               // rows per CTA
-constexpr int RUN = 16;               // score steps (of 64 keys) a CTA takes: 4 to 24 measured, a CTA's start costs about three steps
+constexpr int RUN = 16, RUN_FEW = 8;  // score steps (of 64 keys) a CTA takes; the shorter run where there would be few CTAs (4 to 24
+                                      // measured: a CTA's start costs about three steps)
 constexpr int NS_S = 2, NS_V = 3;     // stages (two CTAs of either kernel share an SM)
 constexpr int BT_CACHE = 512;         // block-table entries kept in shared memory
 constexpr unsigned WAIT_LIMIT = 1u << 26;
@@ -187,7 +188,7 @@ __device__ __forceinline__ int load_keys(const Params& p, const CUtensorMap* map
 // ------------------------------------------------------------------------------------------------------------ scores
 __global__ void __launch_bounds__(64 + EPI * 32, 2) scores_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                                                                      const __grid_constant__ CUtensorMap map_k, const Params p, int n_runs,
-                                                                     int* error) {
+                                                                     int run_steps, int* error) {
   extern __shared__ __align__(1024) unsigned char smem[];
   unsigned char *Qs = smem, *Ks = smem + Q_BYTES;
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + S_TILES + S_STAGE);
@@ -199,7 +200,7 @@ __global__ void __launch_bounds__(64 + EPI * 32, 2) scores_tc_kernel(const __gri
   Tile w;
   if (!find_tile(p, blockIdx.y / n_runs, w)) return;
   const int run = blockIdx.y % n_runs;
-  const int n_steps_all = (w.hi - w.kt0 + BN - 1) / BN, step0 = run * RUN, n_steps = min(n_steps_all - step0, RUN);
+  const int n_steps_all = (w.hi - w.kt0 + BN - 1) / BN, step0 = run * run_steps, n_steps = min(n_steps_all - step0, run_steps);
   if (n_steps <= 0) return;
   if ((smem_u32(smem) & 1023u) != 0) {                        // never seen; refuse rather than compute with a wrong swizzle
     if (threadIdx.x == 0) atomicExch(error, 1);
@@ -519,12 +520,14 @@ int tc_scores(const Params& p, int n_tokens, int max_keys, int max_q, int n_requ
   CUtensorMap map_q, map_k;
   if (int rc = encode_rows(&map_q, p.q, p, n_tokens, D, p.q_stride)) return rc;
   if (int rc = encode_cache(&map_k, p.kc, p)) return rc;
-  const int n_runs = ((max_keys + BN - 1) / BN + RUN - 1) / RUN;
-  const long long y = (long long)row_tiles(p, max_q) * n_runs;
+  const int steps = (max_keys + BN - 1) / BN, tiles = row_tiles(p, max_q);
+  const int run_steps = (long long)tiles * p.G * n_requests * ((steps + RUN - 1) / RUN) >= 3 * sm_count() ? RUN : RUN_FEW;
+  const int n_runs = (steps + run_steps - 1) / run_steps;
+  const long long y = (long long)tiles * n_runs;
   if (y > 65535) return SB_ERR_LIMIT;
   cudaFuncSetAttribute(scores_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, S_SMEM);
   SB_PDL_CHECK(launch_pdl(scores_tc_kernel, dim3(p.G, (unsigned)y, n_requests), dim3(64 + EPI * 32), (size_t)S_SMEM, stream, map_q, map_k, p,
-                          n_runs, error));
+                          n_runs, run_steps, error));
   return 0;
 }
 

@@ -807,7 +807,8 @@ class CudaKernels:
         stats = torch.empty((step, heads, pitch // 64, 2), dtype=torch.float32, device=q.device)
         w = torch.empty((step, heads, pitch), dtype=q.dtype, device=q.device)
         for t0 in range(0, t, step):
-            self.launches += 1 + 2 * ((which & 1) + ((which >> 1) & 1)) if bf16 else 3
+            separate_mix = which & 1 or shape.rows * kv_heads > self.TARGET_BLOCKS      # (else the values' kernel mixes)
+            self.launches += 2 * ((which & 1) + ((which >> 1) & 1)) + (1 if separate_mix else 0) if bf16 else 3
             _check(lib.sb_talking_attention(
                 _p(q), q.stride(0), _p(k_cache), _p(v_cache), _p(block_table), block_table.shape[1], _p(cu_q), _p(kv_len), _p(positions),
                 heads, kv_heads, page_size, k_cache.shape[0], ctypes.c_float(scale), ctypes.c_float(float(softcap or 0.0)), int(chunk or 0),
