@@ -367,12 +367,14 @@ def test_runs_of_tokens_in_a_bounded_scratch_buffer(backend, monkeypatch):
 
 
 @pytest.mark.parametrize("backend", CUDA)
-@pytest.mark.parametrize("heads,kv,dim,chunk,ps", [
-    (8, 2, 64, 100, 32), (32, 8, 128, 0, 32), (5, 1, 48, 64, 32), (40, 2, 16, 130, 32), (16, 4, 128, 65, 16), (6, 2, 64, 0, 256), (4, 4, 64, 64, 8),
-    (12, 1, 128, 150, 64), (34, 2, 64, 90, 128)])
-def test_a_batch_of_unequal_requests_is_each_alone(backend, heads, kv, dim, chunk, ps):
+@pytest.mark.parametrize("heads,kv,dim,chunk,ps,cap,gain", [
+    (8, 2, 64, 100, 32, 8.0, 2.0), (32, 8, 128, 0, 32, 0.0, 2.0), (5, 1, 48, 64, 32, 8.0, 2.0), (40, 2, 16, 130, 32, 100.0, 2.0),
+    (16, 4, 128, 65, 16, 50.0, 1.0), (6, 2, 64, 0, 256, 8.0, 30.0), (4, 4, 64, 64, 8, 100.0, 30.0), (12, 1, 128, 150, 64, 3.0, 2.0),
+    (34, 2, 64, 90, 128, 0.0, 30.0)])
+def test_a_batch_of_unequal_requests_is_each_alone(backend, heads, kv, dim, chunk, ps, cap, gain):
     """The kernels themselves on a batch of decoded tokens, short and long portions (some shapes take the prompts' kernels, some the
-    decoding ones), against the stand-in; and the same rows for every request whatever stands beside it."""
+    decoding ones), against the stand-in; and the same rows for every request whatever stands beside it. Caps that bound every
+    exponential, caps that do not, none; scores far inside a cap, at it, and (gain 30) far beyond what an exponential holds."""
     from serve_b200.engine.step import BatchShape
     from tests.emu_kernels import EmuKernels
 
@@ -413,7 +415,7 @@ def test_a_batch_of_unequal_requests_is_each_alone(backend, heads, kv, dim, chun
         shape = BatchShape(len(rows), len(pos), max(ql), min(ql), max(kl), False, rows_by_q=i32(by_q), neg_q_sorted=tuple(-ql[i] for i in by_q))
         out = torch.full((len(pos), heads * dim), float("nan"), dtype=rt.act_dtype, device=device)
         kernels.talking_attention(qq, kc.to(device), vc.to(device), table[rows].to(device), i32(cu), i32(kl), i32(pos), heads, kv, dim, ps,
-                                  2.0 / dim ** 0.5, talk.to(device), out, shape, chunk=chunk, softcap=8.0, sinks=sinks.to(device))
+                                  gain / dim ** 0.5, talk.to(device), out, shape, chunk=chunk, softcap=cap, sinks=sinks.to(device))
         return out.float().cpu()
 
     every = run(list(range(len(lens))), rt.kernels, dev)
