@@ -2,7 +2,8 @@
 //
 //   sb_add_grouped_rmsnorm  the row is cut into ``groups`` equal parts, each divided by its own sqrt(mean(part^2) + eps), times a
 //                           weight; fused with the residual addition before it and, if asked, with the same kind of norm on the
-//                           sub-layer's output that is added: x += rms_g(a) * w'; out = rms_g(x) * w
+//                           sub-layer's output that is added: x += rms_g(a) * w'; out = rms_g(x) * w. Without a weight out is x
+//                           itself (sub-layers that read the residual stream as it is)
 //   sb_poly_norm            a N(z) + b N(z^2) + c N(z^3) + e, N dividing a row by its root mean square
 //
 // All arithmetic is float; every part of a row is independent of the others, so a block takes one (row, part). Reductions run in a
@@ -32,7 +33,7 @@ __device__ __forceinline__ float dot4(float4 v) { return (v.x * v.x + v.y * v.y)
 __device__ __forceinline__ float4 mul4(float4 v, float f, float4 w) { return make_float4(v.x * f * w.x, v.y * f * w.y, v.z * f * w.z, v.w * f * w.w); }
 
 struct NormArgs {
-  float* x; const void* delta; const float* through; const int* rows; const float* weight; void* out;
+  float* x; const void* delta; const float* through; const int* rows; const float* weight; void* out;      // weight null: out = x
   int dim, part; float eps;        // row length, length of a part
 };
 
@@ -50,9 +51,10 @@ __global__ void __launch_bounds__(512) grouped_norm_vec_kernel(const NormArgs a,
 #pragma unroll
   for (int k = 0; k < VPT; ++k) {        // weights: no kernel of a step writes them
     const int i = at + k * step;
-    w[k] = wd[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+    w[k] = make_float4(1.f, 1.f, 1.f, 1.f);
+    wd[k] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (i < nvec) {
-      w[k] = load4(a.weight + off + i * 4);
+      if (a.weight) w[k] = load4(a.weight + off + i * 4);
       if (a.through) wd[k] = load4(a.through + off + i * 4);
     }
   }
@@ -83,7 +85,7 @@ __global__ void __launch_bounds__(512) grouped_norm_vec_kernel(const NormArgs a,
     v[k].x += d[k].x; v[k].y += d[k].y; v[k].z += d[k].z; v[k].w += d[k].w;
     ss += dot4(v[k]);
   }
-  const float inv = 1.0f / sqrtf(sum(ss) / (float)a.part + a.eps);
+  const float inv = a.weight ? 1.0f / sqrtf(sum(ss) / (float)a.part + a.eps) : 1.0f;
   TO* orow = (TO*)a.out + (size_t)r * a.dim + off;
 #pragma unroll
   for (int k = 0; k < VPT; ++k) {
@@ -121,12 +123,12 @@ __global__ void __launch_bounds__(256) grouped_norm_kernel(const NormArgs a) {
     buf[i] = v;
     ss += v * v;
   }
-  const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)a.part + a.eps);
+  const float inv = a.weight ? 1.0f / sqrtf(block_sum(ss, red) / (float)a.part + a.eps) : 1.0f;
   TO* orow = (TO*)a.out + (size_t)blockIdx.x * a.dim + off;
   for (int i = threadIdx.x; i < a.part; i += blockDim.x) {
     const float v = buf[i];
     if (xr && dr && !a.rows) xr[i] = v;
-    orow[i] = from_float<TO>(v * inv * a.weight[off + i]);
+    orow[i] = from_float<TO>(a.weight ? v * inv * a.weight[off + i] : v);
   }
 }
 
@@ -249,11 +251,11 @@ __global__ void __launch_bounds__(256) poly_norm_kernel(const T* z, const float*
 }  // namespace
 
 // x float [*, dim] or null; delta [*, dim] of delta_dtype or null; through float [dim] or null (the weight of the norm the delta goes
-// through first); rows int [n_rows] or null (only these rows, x stays as it is); weight float [dim]; out [n_rows, dim] of out_dtype.
+// through first); rows int [n_rows] or null (only these rows, x stays as it is); weight float [dim], or null: no second norm; out [n_rows, dim] of out_dtype.
 SB_EXPORT int sb_add_grouped_rmsnorm(float* x, const void* delta, int delta_dtype, const float* through, const int* rows, const float* weight,
                                      void* out, int out_dtype, int n_rows, int dim, int groups, float eps, cudaStream_t stream) {
   if (n_rows <= 0) return 0;
-  if (dim <= 0 || groups <= 0 || dim % groups || groups > 65535 || !weight || !out || (!x && !delta) || (through && !delta)) return SB_ERR_SHAPE;
+  if (dim <= 0 || groups <= 0 || dim % groups || groups > 65535 || !out || (!x && !delta) || (through && !delta)) return SB_ERR_SHAPE;
   const bool df = delta == nullptr || delta_dtype == SB_DTYPE_F32;
   if (!df && delta_dtype != SB_DTYPE_BF16) return SB_ERR_DTYPE;
   const NormArgs a = {x, delta, through, rows, weight, out, dim, dim / groups, eps};

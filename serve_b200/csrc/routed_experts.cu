@@ -88,12 +88,14 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict_
 // As moe_route_kernel, for a router with a bias on the choice: the scores (softmax over the first E of a row's ``stride``
 // logits, or sigmoid) choose through score + bias[e], lowest index first on ties, while the weights are the scores
 // themselves, divided by (their sum + sum_eps) if asked. A lane holds PER_LANE outputs (E <= 32 * PER_LANE): few for the
-// usual counts, so the loops over them are short. E counts every output the router scores; an index at or beyond
+// usual counts, so the loops over them are short. With n_groups > 1 the E outputs form as many equal groups of neighbours;
+// a group is as good as its best output, and only outputs of the keep_groups best groups can be chosen. E counts every output the router scores; an index at or beyond
 // the number of real experts means "the token itself" to the kernels after this one.
 template <int PER_LANE>
 __global__ void __launch_bounds__(128) moe_route_bias_kernel(const float* __restrict__ logits, int stride, int E, int top, int score_kind,
                                                              int renorm, float sum_eps, const float* __restrict__ bias, int n_tokens,
-                                                             int* __restrict__ idx, float* __restrict__ wts, float weight_scale) {
+                                                             int* __restrict__ idx, float* __restrict__ wts, float weight_scale,
+                                                             int n_groups, int keep_groups) {
   const int lane = threadIdx.x & 31;
   const int t = blockIdx.x * 4 + (threadIdx.x >> 5);
   if (t >= n_tokens) return;
@@ -126,6 +128,32 @@ __global__ void __launch_bounds__(128) moe_route_bias_kernel(const float* __rest
   for (int u = 0; u < PER_LANE; ++u) {
     const int e = lane + 32 * u;
     pick[u] = e < E ? score[u] + (bias ? bias[e] : 0.f) : -INFINITY;
+  }
+  if (keep_groups < n_groups) {
+    // the best output of those in no kept group yet names the next group to keep
+    const int gs = E / n_groups;
+    unsigned kept = 0;                          // bit u: this lane's output lane + 32 u is in a kept group
+    for (int s = 0; s < keep_groups; ++s) {
+      float m = -INFINITY;
+      int arg = 0x7fffffff;
+#pragma unroll
+      for (int u = 0; u < PER_LANE; ++u) {
+        const int e = lane + 32 * u;
+        if (e < E && !((kept >> u) & 1u) && (pick[u] > m || (pick[u] == m && e < arg))) { m = pick[u]; arg = e; }
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float om = __shfl_xor_sync(0xffffffffu, m, o);
+        const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
+        if (om > m || (om == m && oa < arg)) { m = om; arg = oa; }
+      }
+#pragma unroll
+      for (int u = 0; u < PER_LANE; ++u)
+        if ((lane + 32 * u) / gs == arg / gs) kept |= 1u << u;
+    }
+#pragma unroll
+    for (int u = 0; u < PER_LANE; ++u)
+      if (!((kept >> u) & 1u)) pick[u] = -INFINITY;
   }
   float val = 0.f, total = 0.f;                 // lane s keeps the s-th choice
   int chosen = 0;
@@ -825,16 +853,20 @@ SB_EXPORT int sb_moe_combine(const float* parts, int top, int n_tokens, int N, v
 }
 
 // As sb_moe_route with more: the row stride of the logits (columns beyond E are not the router's), a float bias [E] or
-// null that joins the scores for the choice only, sum_eps, added to the sum the chosen scores are divided by, and
-// weight_scale, a constant every weight is multiplied by.
+// null that joins the scores for the choice only, sum_eps, added to the sum the chosen scores are divided by,
+// weight_scale, a constant every weight is multiplied by, and n_groups equal groups of outputs of which only the keep_groups
+// best are open to the choice (1, 1: all are).
 SB_EXPORT int sb_moe_route_bias(const float* logits, int stride, int E, int top, int score_kind, int renorm, float sum_eps,
-                                const float* bias, int n_tokens, int* idx, float* wts, float weight_scale, cudaStream_t stream) {
+                                const float* bias, int n_tokens, int* idx, float* wts, float weight_scale, int n_groups, int keep_groups,
+                                cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   if (E <= 0 || top <= 0 || top > E || top > ROUTE_MAX_TOP || E > 32 * ROUTE_PER_LANE) return SB_ERR_LIMIT;
   if (stride < E) return SB_ERR_SHAPE;
+  if (n_groups <= 0 || E % n_groups || keep_groups <= 0 || keep_groups > n_groups || (long long)top > (long long)keep_groups * (E / n_groups)) return SB_ERR_SHAPE;
   auto k = E <= 64 ? moe_route_bias_kernel<2> : E <= 128 ? moe_route_bias_kernel<4> : E <= 256 ? moe_route_bias_kernel<8>
                                                                                                : moe_route_bias_kernel<ROUTE_PER_LANE>;
-  k<<<(n_tokens + 3) / 4, 128, 0, stream>>>(logits, stride, E, top, score_kind, renorm, sum_eps, bias, n_tokens, idx, wts, weight_scale);
+  k<<<(n_tokens + 3) / 4, 128, 0, stream>>>(logits, stride, E, top, score_kind, renorm, sum_eps, bias, n_tokens, idx, wts, weight_scale,
+                                            n_groups, keep_groups);
   SB_LAUNCH_CHECK();
   return 0;
 }

@@ -157,9 +157,11 @@ __global__ void __launch_bounds__(CONV_THREADS) conv_state_kernel(const T* __res
 // tokens' vectors come through a two-stage cp.async ring, REC_TS tokens a stage, so the next tokens arrive while
 // these are worked on; a thread's rows are 4 P apart in fours, so it reads them 16 bytes at a time and the lanes of
 // a column read neighbouring 16 bytes.
-constexpr int MODE_DECAY = 0, MODE_SSM = 1, MODE_DELTA = 2, MODE_WKV = 3, MODE_GLA = 4;
+constexpr int MODE_DECAY = 0, MODE_SSM = 1, MODE_DELTA = 2, MODE_WKV = 3, MODE_GLA = 4, MODE_RET = 5;
 // MODE_GLA: S <- diag(a) S + k v^T, o = S^T q (read out after the update), a = sigmoid(rate + bias)^rate_scale per row of S,
 // formed as exp(-softplus(-(rate + bias)) * rate_scale); q times q_scale.
+// MODE_RET: MODE_DECAY's update with q, k and v as projected, the first rot_dims elements of q and k rotated by position (pairs
+// i, i + rot_dims / 2), k times k_scale.
 constexpr int REC_RPT = 16;
 constexpr int REC_THREADS = 128;
 constexpr int REC_TS = 16;
@@ -180,6 +182,9 @@ struct RecArgs {
   float* out; int out_stride;                        // [T, H * dv] float
   int H, Hqk, dk, dv, P, dkp, dvp, n_tokens;
   float q_scale;
+  const int* positions; const float* inv_freq;       // RET: [T] and [rot_dims / 2]
+  int rot_dims;
+  float k_scale;
   float rate_scale;                                  // GLA: the exponent of the sigmoid (one over the temperature)
   // float work space, made by the first kernel: qf, kf [T, Hqk, dkp]; af [T, H, dkp] (DELTA, WKV, GLA); vf [T, H, dvp]; sc, dec [T, H]
   float *qf, *kf, *af, *vf, *sc, *dec;
@@ -212,7 +217,23 @@ __global__ void __launch_bounds__(REC_THREADS) recurrence_prep_kernel(RecArgs a)
       fk = 1.f / sqrtf(sk + 1e-6f);
     }
     if (MODE == MODE_GLA) fq = a.q_scale;
-    for (int i = tid; i < dkp; i += 32) {
+    int i0 = 0;
+    if (MODE == MODE_RET) {
+      fk = a.k_scale;
+      i0 = a.rot_dims;
+      const int half = a.rot_dims >> 1;
+      const float pos = (float)a.positions[t];
+      for (int i = tid; i < half; i += 32) {
+        float s, c;
+        sincosf(pos * a.inv_freq[i], &s, &c);
+        const float qu = to_float(qr[i]), qv = to_float(qr[i + half]), ku = to_float(kr[i]), kv = to_float(kr[i + half]);
+        qo[i] = qu * c - qv * s;
+        qo[i + half] = qv * c + qu * s;
+        ko[i] = (ku * c - kv * s) * fk;
+        ko[i + half] = (kv * c + ku * s) * fk;
+      }
+    }
+    for (int i = i0 + tid; i < dkp; i += 32) {
       float x = 0.f, y = 0.f;
       if (i < dk) {
         x = to_float(qr[i]);
@@ -267,7 +288,7 @@ __global__ void __launch_bounds__(REC_THREADS) recurrence_prep_kernel(RecArgs a)
     }
     if (tid == 0) {
       float sc = 1.f, dec = 1.f;
-      if (MODE == MODE_DECAY) dec = ((const float*)a.decay)[h];
+      if (MODE == MODE_DECAY || MODE == MODE_RET) dec = ((const float*)a.decay)[h];
       if (MODE == MODE_SSM) {
         sc = softplus_f(to_float(((const T*)a.aux)[(size_t)t * a.aux_stride + h]) + load_w(a.dt_bias, a.par_dtype, h));
         dec = expf(-expf(load_w(a.a_log, a.par_dtype, h)) * sc);
@@ -456,7 +477,7 @@ int launch_recurrence(RecArgs a, float* work, int n_rows, cudaStream_t stream) {
   const int per_tok = ((MODE == MODE_DELTA || MODE == MODE_WKV || MODE == MODE_GLA) ? 3 : 2) * a.dkp + VC;
   const size_t smem = (size_t)2 * (REC_TS * per_tok + 2 * REC_TS) * sizeof(float);
   dim3 grid(a.dvp / VC, a.H, n_rows);
-  auto kernel = recurrence_scan_kernel<MODE>;
+  auto kernel = recurrence_scan_kernel<MODE == MODE_RET ? MODE_DECAY : MODE>;      // (they differ in what the first kernel leaves)
   if (smem > 48 * 1024) {
     if (smem > 200 * 1024) return SB_ERR_LIMIT;
     cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -756,7 +777,8 @@ SB_EXPORT long long sb_linear_recurrence_work_floats(int mode, int n_tokens, int
 
 // The recurrences (mode 0: fixed decay per head with silu on q, k, v; 1: selective state space; 2: gated delta rule, its
 // rate per row of the state or, with rate_per_head, per head; 3: decay per key channel with a bonus [H, dk] for the
-// current token, read out before the update). See RecArgs for what each pointer is; unused ones are null. ``rate`` has a
+// current token, read out before the update; 4: decay per key channel, read out after it; 5: fixed decay per head on q, k, v as
+// projected, q and k rotated by ``positions`` and ``inv_freq``, k times k_scale). See RecArgs for what each pointer is; unused ones are null. ``rate`` has a
 // dtype of its own (rate_dtype). out is float [T, H * dv]; work: 16-byte aligned floats,
 // as many as sb_linear_recurrence_work_floats says.
 SB_EXPORT int sb_linear_recurrence(int mode, const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride,
@@ -764,13 +786,14 @@ SB_EXPORT int sb_linear_recurrence(int mode, const void* q, int q_stride, const 
                                    const float* bonus, const float* decay, const void* a_log, const void* dt_bias, const void* d_skip, int par_dtype, float* state,
                                    const int* slots, const int* cu_q, float* out, int out_stride, int H, int Hqk, int dk, int dv,
                                    float q_scale, int n_rows, int n_tokens, float* work, long long state_stride, int dtype, float rate_scale,
-                                   cudaStream_t stream) {
+                                   const int* positions, const float* inv_freq, int rot_dims, float k_scale, cudaStream_t stream) {
   if (n_rows <= 0 || n_tokens <= 0) return 0;
   if (!work || !aligned16(work)) return SB_ERR_ALIGN;
   if (H <= 0 || Hqk <= 0 || H % Hqk || dk <= 0 || dv <= 0) return SB_ERR_SHAPE;
   if (n_rows > 65535 || H > 65535 || dk > 32 * REC_RPT) return SB_ERR_LIMIT;
   if (mode == MODE_WKV && (H != Hqk || !rate || !dt_bias || !bonus)) return SB_ERR_SHAPE;
   if (mode == MODE_GLA && (!rate || !dt_bias)) return SB_ERR_SHAPE;
+  if (mode == MODE_RET && (H != Hqk || !decay || rot_dims < 0 || (rot_dims & 1) || rot_dims > dk || (rot_dims && (!positions || !inv_freq)))) return SB_ERR_SHAPE;
   if (rate && rate_dtype != SB_DTYPE_F32 && rate_dtype != SB_DTYPE_BF16) return SB_ERR_DTYPE;
   RecArgs a;
   a.q = q; a.k = k; a.v = v; a.q_stride = q_stride; a.k_stride = k_stride; a.v_stride = v_stride;
@@ -778,6 +801,7 @@ SB_EXPORT int sb_linear_recurrence(int mode, const void* q, int q_stride, const 
   a.rate_per_head = rate_per_head; a.bonus = bonus; a.decay = decay;
   a.a_log = a_log; a.dt_bias = dt_bias; a.d_skip = d_skip; a.par_dtype = par_dtype; a.state = state; a.state_stride = state_stride; a.slots = slots; a.cu_q = cu_q;
   a.out = out; a.out_stride = out_stride; a.H = H; a.Hqk = Hqk; a.dk = dk; a.dv = dv; a.P = 1; a.dkp = a.dvp = 0; a.n_tokens = n_tokens;
+  a.positions = positions; a.inv_freq = inv_freq; a.rot_dims = rot_dims; a.k_scale = k_scale;
   a.q_scale = q_scale; a.rate_scale = rate_scale; a.qf = a.kf = a.af = a.vf = a.sc = a.dec = nullptr;
   if (dtype == SB_DTYPE_F32) {
     if (mode == MODE_DECAY) return launch_recurrence<float, MODE_DECAY>(a, work, n_rows, stream);
@@ -785,12 +809,14 @@ SB_EXPORT int sb_linear_recurrence(int mode, const void* q, int q_stride, const 
     if (mode == MODE_DELTA) return launch_recurrence<float, MODE_DELTA>(a, work, n_rows, stream);
     if (mode == MODE_WKV) return launch_recurrence<float, MODE_WKV>(a, work, n_rows, stream);
     if (mode == MODE_GLA) return launch_recurrence<float, MODE_GLA>(a, work, n_rows, stream);
+    if (mode == MODE_RET) return launch_recurrence<float, MODE_RET>(a, work, n_rows, stream);
   } else if (dtype == SB_DTYPE_BF16) {
     if (mode == MODE_DECAY) return launch_recurrence<__nv_bfloat16, MODE_DECAY>(a, work, n_rows, stream);
     if (mode == MODE_SSM) return launch_recurrence<__nv_bfloat16, MODE_SSM>(a, work, n_rows, stream);
     if (mode == MODE_DELTA) return launch_recurrence<__nv_bfloat16, MODE_DELTA>(a, work, n_rows, stream);
     if (mode == MODE_WKV) return launch_recurrence<__nv_bfloat16, MODE_WKV>(a, work, n_rows, stream);
     if (mode == MODE_GLA) return launch_recurrence<__nv_bfloat16, MODE_GLA>(a, work, n_rows, stream);
+    if (mode == MODE_RET) return launch_recurrence<__nv_bfloat16, MODE_RET>(a, work, n_rows, stream);
   } else {
     return SB_ERR_DTYPE;
   }

@@ -367,8 +367,9 @@ class CudaKernels:
     def add_grouped_rmsnorm(self, x, delta, through, rows, weight, groups: int, eps: float, out) -> None:
         """x += d; out = every one of ``groups`` equal parts of x divided by its own root mean square, times weight (float). d is
         ``delta`` (activations or float), or, with ``through`` (the float weight of such a norm the delta still has to pass), that
-        norm of it. With ``rows`` only those rows, and x stays as it is; with x None, out = the norm of delta."""
-        if weight.dtype != torch.float32 or (through is not None and through.dtype != torch.float32):
+        norm of it. With ``rows`` only those rows, and x stays as it is; with x None, out = the norm of delta. ``weight`` None: out =
+        x as it is (after the addition)."""
+        if (weight is not None and weight.dtype != torch.float32) or (through is not None and through.dtype != torch.float32):
             raise KernelError("add_grouped_rmsnorm: the weights are float")
         self.launches += 1
         n_rows = rows.shape[0] if rows is not None else out.shape[0]
@@ -517,13 +518,14 @@ class CudaKernels:
 
     def latent_prepare(self, proj, n_q, positions, token_row, c_weight, eps, inv_freq, rot_dims, heads, dim, rot_dim, rank, head_dim,
                        q_lat, k_cache, block_table, page_size, write_cache, q_off=None, row_out=None,
-                       half_pairs: bool = False, latent=None) -> None:
+                       half_pairs: bool = False, latent=None, rot_mult: float = 1.0) -> None:
         """Latent attention between its input product and its attention: proj [T, >= n_q + rank + rot_dim] holds the heads'
         queries ([dim | rot_dim] each), the latent vector and the shared key part. Writes the cache row [normed latent | rotated
         key part | zeros] (if write_cache), the same row into row_out [T, >= rank + rot_dim] (if given), and columns
         [q_off, head_dim) of every head of q_lat (rotated query part, zeros); q_off defaults to rank. Rotated pairs are
         (2 i, 2 i + 1), or with ``half_pairs`` (i, i + rot_dims / 2). ``latent`` [T, >= rank + rot_dim]: the latent vector and the shared
-        key part in a buffer of their own (proj then holds the queries only)."""
+        key part in a buffer of their own (proj then holds the queries only). Cosines and sines are multiplied by ``rot_mult``. With
+        neither write_cache nor row_out there is no latent vector: only the queries are prepared (c_weight may be None)."""
         self.launches += 1
         pages = k_cache.shape[0] if k_cache is not None else 0
         _check(self._prep_lib().sb_latent_prepare(
@@ -531,7 +533,7 @@ class CudaKernels:
             dim, rot_dim, rank, head_dim, _p(q_lat), q_lat.stride(0), rank if q_off is None else q_off, _p(row_out),
             row_out.stride(0) if row_out is not None else 0, _p(k_cache), _p(block_table), block_table.shape[1], page_size, pages,
             1 if write_cache else 0, _p(self.errors_tensor()), proj.shape[0], _DT[proj.dtype], 1 if half_pairs else 0, _p(latent),
-            latent.stride(0) if latent is not None else 0, self._s()),
+            latent.stride(0) if latent is not None else 0, ctypes.c_float(rot_mult), self._s()),
             "latent attention preparation")
 
     def linear(self, a, w, out) -> None:
@@ -1019,18 +1021,20 @@ class CudaKernels:
 
     def linear_recurrence(self, mode: str, q, k, v, state, ctx, out, heads: int, qk_heads: int, dk: int, dv: int, aux=None, rate=None,
                           decay=None, a_log=None, dt_bias=None, d_skip=None, q_scale: float = 1.0, rate_per_head: bool = False,
-                          bonus=None, rate_scale: float = 1.0) -> None:
+                          bonus=None, rate_scale: float = 1.0, inv_freq=None, rot_dims: int = 0, k_scale: float = 1.0) -> None:
         """One matrix state [dk, dv] per (request, head), walked over the step's tokens: see csrc/sequence_ops.cu.
         mode "decay": S = decay_h S + k v^T with silu on q, k, v; "ssm": S = exp(-exp(a_log) dt) S + dt k v^T, dt =
         softplus(aux + dt_bias), o += d_skip v; "delta": S = g S, S += k (beta (v - S^T k))^T with g = exp(-exp(a_log)
         softplus(rate + dt_bias)), beta = sigmoid(aux), q and k made unit vectors (``rate_per_head``: rate [T, heads] and dt_bias
         [heads], one decay for a head's whole state); "wkv": o = S^T q + (sum_i q_i bonus_i k_i) v, then S = diag(d) S + k v^T
         with d = exp(-exp(rate + dt_bias)) per row (rate [T, heads * dk], of a dtype of its own; bonus float [heads * dk]);
-        "gla": S = diag(a) S + k v^T, o = S^T (q_scale q), a = sigmoid(rate + dt_bias)^rate_scale per row (rate [T, heads * dk]).
+        "gla": S = diag(a) S + k v^T, o = S^T (q_scale q), a = sigmoid(rate + dt_bias)^rate_scale per row (rate [T, heads * dk]);
+        "retention": S = decay_h S + k v^T on q, k, v as they are, the first rot_dims elements of q and k rotated by the tokens'
+        positions (pairs i, i + rot_dims / 2; inv_freq float [rot_dims / 2]), k times k_scale.
         out: float [T, heads * dv]."""
         par = a_log if a_log is not None else (dt_bias if mode == "gla" else None)
         lib = self._seq_lib()
-        code = {"decay": 0, "ssm": 1, "delta": 2, "wkv": 3, "gla": 4}[mode]
+        code = {"decay": 0, "ssm": 1, "delta": 2, "wkv": 3, "gla": 4, "retention": 5}[mode]
         lib.sb_linear_recurrence_work_floats.restype = ctypes.c_longlong
         need = lib.sb_linear_recurrence_work_floats(code, q.shape[0], heads, qk_heads, dk, dv)
         if need < 0:
@@ -1043,8 +1047,8 @@ class CudaKernels:
             _DT[rate.dtype] if rate is not None else 0, 1 if rate_per_head else 0, _p(bonus), _p(decay),
             _p(a_log), _p(dt_bias), _p(d_skip), _DT[par.dtype] if par is not None else 0, _p(state), _p(ctx.slots), _p(ctx.cu_q),
             _p(out), out.stride(0), heads, qk_heads, dk, dv, ctypes.c_float(q_scale), ctx.shape.rows, q.shape[0], _p(work),
-            ctypes.c_longlong(state.stride(0)), _DT[v.dtype], ctypes.c_float(rate_scale), self._s()),
-            "linear recurrence")
+            ctypes.c_longlong(state.stride(0)), _DT[v.dtype], ctypes.c_float(rate_scale), _p(ctx.positions), _p(inv_freq), int(rot_dims),
+            ctypes.c_float(k_scale), self._s()), "linear recurrence")
 
     def gated_norm(self, y, out, groups: int = 0, eps: float = 0.0, weight=None, gate=None, gate_act: str = "sigmoid",
                    gate_first: bool = False, scale: float = 1.0) -> None:
@@ -1070,12 +1074,13 @@ class CudaKernels:
     def routed_experts(self, h, logits, w_gate_up, w_down, top: int, out, score: str = "sigmoid", renormalise: bool = False,
                        scale_input: bool = True, activation: str = "clamped_swish", limit: float = 0.0, alpha: float = 1.702,
                        outputs=None, choice_bias=None, renormalise_eps: float = 0.0, shared=None, shared_gated: bool = False,
-                       weight_scale: float = 1.0) -> None:
+                       weight_scale: float = 1.0, groups: int = 1, keep_groups: int = 1) -> None:
         """out[t] = sum over the ``top`` best experts e of expert_e(w_e * h[t]) (or w_e * expert_e(h[t])): logits float [T, E],
         w_gate_up [E, 2 ff, K], w_down [E, N, ff]. More: the router scores the first ``outputs`` columns of logits, of which those
         beyond the E experts stand for the token's input itself; ``choice_bias`` (float [outputs]) joins the scores for the choice
         only; ``renormalise_eps`` joins the sum the weights are divided by; ``shared`` [T, N] is added for every token, times
-        sigmoid(logits[:, outputs]) if ``shared_gated``; every weight is multiplied by ``weight_scale``."""
+        sigmoid(logits[:, outputs]) if ``shared_gated``; every weight is multiplied by ``weight_scale``; only outputs of the
+        ``keep_groups`` best of ``groups`` equal groups of neighbours can be chosen (a group is as good as its best output)."""
         lib = self._moe_lib()
         t = logits.shape[0]
         e = w_down.shape[0]
@@ -1101,7 +1106,7 @@ class CudaKernels:
         if more:
             _check(lib.sb_moe_route_bias(_p(logits), logits.stride(0), outputs, top, {"sigmoid": 0, "softmax": 1}[score],
                                          1 if renormalise else 0, ctypes.c_float(renormalise_eps), _p(choice_bias), t, _p(idx), _p(wts),
-                                         ctypes.c_float(weight_scale), s), "expert choice")
+                                         ctypes.c_float(weight_scale), int(groups), int(keep_groups), s), "expert choice")
         else:
             _check(lib.sb_moe_route(_p(logits), e, top, {"sigmoid": 0, "softmax": 1}[score], 1 if renormalise else 0, t, _p(idx), _p(wts), s),
                    "expert choice")

@@ -10,6 +10,8 @@ All of them keep S [dk, dv] per (request, head) in float and differ in how a tok
   "wkv"          o = (S + diag(u_h) k v^T)^T r;  S <- diag(d) S + k v^T      r, k, v, the gate and the decay each read
                  their own blend of the token's input with the one before; d = exp(-exp(w0 + W2 tanh(W1 x_w))) per key
                  channel; the bonus u_h counts for the current token only, and the read-out comes before the update
+  "retention"    S <- decay_h S + k v^T,  o = S^T q          q, k, v as projected, q and k rotated by position, k times dk^-1/2;
+                 decay_h fixed per head
   "gated_linear_attention"  S <- diag(a) S + k v^T,  o = S^T q      q times dk^-1/2; a = sigmoid(W_a2 (W_a1 h) + b)^(1/tau) per key
                  channel, formed in float as exp(log_sigmoid(z) / tau); the read-out comes after the update
 
@@ -25,6 +27,7 @@ import torch
 
 from ..config.spec import PartSpec
 from .base import CacheNeed, Mixer, TensorDecl, build_part, register_part
+from .rotary import PAIRING_HALF
 
 
 class RecurrentMixer(Mixer):
@@ -94,6 +97,56 @@ class LightningMixer(RecurrentMixer):
         y = self._readout(t)
         k.linear_recurrence("decay", proj[:, :hk], proj[:, hk: 2 * hk], proj[:, 2 * hk: 2 * hk + hv], cache.states["state"], ctx, y,
                             self.heads, self.heads, self.dim, self.vdim, decay=self.decay)
+        self.norm.forward(y, proj[:, 2 * hk + hv:], out, scale)
+
+
+@register_part("mixer", "retention")
+class RetentionMixer(RecurrentMixer):
+    """params: hidden, heads, dim, vdim, decay (one per head), eps, position (a PartSpec: rotary in the half layout, or none).
+    Tensors: "q", "k" [heads * dim, hidden], "v", "g" [heads * vdim, hidden], "o". The read-out is divided by its root mean
+    square per head, without a weight, and multiplied by silu(W_g h)."""
+
+    def __init__(self, spec, runtime):
+        super().__init__(spec, runtime)
+        p = spec.params
+        self._common(p)
+        self.dim, self.vdim = int(p["dim"]), int(p["vdim"])
+        self.decay_values = [float(d) for d in p["decay"]]
+        if len(self.decay_values) != self.heads:
+            raise ValueError(f"{len(self.decay_values)} decays for {self.heads} heads")
+        self.position = build_part("position", p.get("position") or PartSpec("none"), runtime)
+        if self.position.rotary_dim and (self.position.pairing != PAIRING_HALF or self.position.rotary_dim > self.dim):
+            raise ValueError("retention: the rotation pairs elements i and i + rotary_dim / 2 of the first rotary_dim of a head")
+        self.mixed_size = self.heads * self.vdim
+        self.norm = build_part("norm", PartSpec("gated_group_rms", {"channels": self.mixed_size, "groups": self.heads, "eps": self.eps,
+                                                                    "weight_name": None, "gate": "silu"}, self.prefix), runtime)
+
+    def kernel_needs(self):
+        return {"libraries": ["seq"]}
+
+    def tensor_decls(self):
+        hk, hv = self.heads * self.dim, self.heads * self.vdim
+        return [TensorDecl(self._name("q"), (hk, self.hidden)), TensorDecl(self._name("k"), (hk, self.hidden)),
+                TensorDecl(self._name("v"), (hv, self.hidden)), TensorDecl(self._name("g"), (hv, self.hidden)),
+                TensorDecl(self._name("o"), (self.hidden, hv))]
+
+    def load(self, tensors):
+        self.w_in = torch.cat([tensors[self._name(n)] for n in ("q", "k", "v", "g")], dim=0).contiguous()
+        self.w_o = tensors[self._name("o")].contiguous()
+        self.decay = torch.tensor(self.decay_values, dtype=torch.float32, device=self.w_o.device)
+
+    def cache_need(self):
+        return CacheNeed(states=(("state", (self.heads, self.dim, self.vdim)),))
+
+    def mix_into(self, h, ctx, cache, out, scale: float = 1.0):
+        k = self.rt.kernels
+        t, hk, hv = h.shape[0], self.heads * self.dim, self.heads * self.vdim
+        proj = self.rt.empty_act((t, 2 * hk + 2 * hv))
+        k.linear(h, self.w_in, proj)
+        y = self._readout(t)
+        k.linear_recurrence("retention", proj[:, :hk], proj[:, hk: 2 * hk], proj[:, 2 * hk: 2 * hk + hv], cache.states["state"], ctx, y,
+                            self.heads, self.heads, self.dim, self.vdim, decay=self.decay, inv_freq=self.position.inv_freq,
+                            rot_dims=self.position.rotary_dim, k_scale=1.0 / math.sqrt(self.dim))
         self.norm.forward(y, proj[:, 2 * hk + hv:], out, scale)
 
 

@@ -80,9 +80,9 @@ class LayerNorm(RMSNorm):
 class GroupedRMSNorm(Norm):
     """The vector is cut into ``groups`` equal consecutive parts, each divided by its own sqrt(mean(part^2) + eps); then a weight
     per element. ``scale_name``: a second factor per element (a layer scale behind a norm after a sub-layer), multiplied into the
-    weight at load in float. The same fusion with the residual addition as the other norms; and the norm of the sub-layer before
+    weight at load in float; ``multiplier``: a constant factor, likewise. The same fusion with the residual addition as the other norms; and the norm of the sub-layer before
     (a ``DeferredNorm`` of this kind with the same parts) is applied in the same kernel: x += n'(a); y = n(x).
-    params: size, groups, eps, weight_name, scale_name."""
+    params: size, groups, eps, weight_name, scale_name, multiplier."""
 
     def __init__(self, spec, runtime):
         super().__init__(spec, runtime)
@@ -92,6 +92,7 @@ class GroupedRMSNorm(Norm):
             raise ValueError(f"grouped_rms: {self.size} elements cannot be cut into {self.groups} equal parts")
         self.weight_name = self.prefix + p.get("weight_name", "weight")
         self.scale_name = self.prefix + p["scale_name"] if p.get("scale_name") else None
+        self.multiplier = float(p["multiplier"]) if p.get("multiplier") is not None else 1.0
         self.weight = None
 
     def kernel_needs(self):
@@ -105,6 +106,8 @@ class GroupedRMSNorm(Norm):
         w = tensors[self.weight_name].float()
         if self.scale_name:
             w = w * tensors[self.scale_name].float()
+        if self.multiplier != 1.0:
+            w = w * self.multiplier
         self.weight = w.contiguous()
 
     def _split(self, delta):
@@ -134,6 +137,41 @@ class GroupedRMSNorm(Norm):
         out = torch.empty((a.shape[0], self.size), dtype=torch.float32, device=a.device)
         self.rt.kernels.add_grouped_rmsnorm(None, a, None, None, self.weight, self.groups, self.eps, out)
         return out
+
+
+@register_part("norm", "identity")
+class IdentityNorm(Norm):
+    """No norm at all: what a sub-layer that reads the residual stream as it is has in front of it. The pending delta is added in
+    the same kernel that rounds the stream to the activations' type, and so is the norm of the sub-layer before, if that is a
+    ``grouped_rms``: x += n'(a); y = x. params: size."""
+
+    def __init__(self, spec, runtime):
+        super().__init__(spec, runtime)
+        self.size = int(spec.params["size"])
+
+    def kernel_needs(self):
+        return {"libraries": ["prep"]}
+
+    @staticmethod
+    def _split(delta):
+        """(tensor to add or None, the ``grouped_rms`` it goes through first or None)."""
+        if isinstance(delta, DeferredNorm):
+            return (delta.a, delta.norm) if isinstance(delta.norm, GroupedRMSNorm) else (delta.plain(), None)
+        return plain_delta(delta), None
+
+    def _run(self, x, delta, rows, out):
+        a, n = self._split(delta)
+        self.rt.kernels.add_grouped_rmsnorm(x, a, n.weight if n else None, rows, None, n.groups if n else 1, n.eps if n else 0.0, out)
+        return out
+
+    def forward(self, x, delta, ctx):
+        return self._run(x, delta, None, self.rt.empty_act((x.shape[0], self.size)))
+
+    def forward_rows(self, x, delta, rows, ctx):
+        return self._run(x, delta, rows, self.rt.empty_act((rows.shape[0], self.size)))
+
+    def apply(self, a):
+        return a.float()
 
 
 @register_part("norm", "dynamic_tanh")

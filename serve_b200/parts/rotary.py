@@ -24,14 +24,28 @@ def rotary_inv_freq(rotary_dim: int, theta: float, scaling=None) -> torch.Tensor
     """float32 [rotary_dim/2] inverse frequencies, scaled per frequency if asked.
 
     ``scaling`` is None, a mapping with factor, low_freq_factor,
-    high_freq_factor, original_max_position_embeddings (the llama3 rule), or
-    {"kind": "linear", "factor": f}: every frequency divided by f.
+    high_freq_factor, original_max_position_embeddings (the llama3 rule),
+    {"kind": "linear", "factor": f}: every frequency divided by f, or
+    {"kind": "yarn", "factor", "original", "fast", "slow"} (YaRN, Peng et al.): pair i
+    keeps 1 - r_i of its frequency and takes r_i of it divided by the factor, r a ramp
+    over i from the pair that turns ``fast`` times in ``original`` positions to the one
+    that turns ``slow`` times (``rotary_length`` says how much longer the rotated
+    vectors get).
     """
     freqs = 1.0 / (theta ** (torch.arange(0, rotary_dim, 2)[: rotary_dim // 2].float() / rotary_dim))
     if scaling is None:
         return freqs
     if scaling.get("kind") == "linear":
         return (freqs / float(scaling["factor"])).to(torch.float32)
+    if scaling.get("kind") == "yarn":
+        factor, original = float(scaling["factor"]), float(scaling["original"])
+        pair = lambda turns: rotary_dim * math.log(original / (2 * math.pi * turns)) / (2 * math.log(theta))
+        lo = max(math.floor(pair(float(scaling["fast"]))), 0)
+        hi = min(math.ceil(pair(float(scaling["slow"]))), rotary_dim - 1)
+        i = torch.arange(rotary_dim // 2, dtype=torch.float64)
+        ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+        f = theta ** (-2.0 * i / rotary_dim)
+        return (f / factor * ramp + f * (1.0 - ramp)).to(torch.float32)
     factor = float(scaling["factor"])
     low = float(scaling["low_freq_factor"])
     high = float(scaling["high_freq_factor"])
@@ -51,6 +65,13 @@ def rotary_inv_freq(rotary_dim: int, theta: float, scaling=None) -> torch.Tensor
     return torch.stack([torch.as_tensor(v, dtype=torch.float32) for v in out]).to(torch.float32)
 
 
+def rotary_length(scaling=None) -> float:
+    """What cosines and sines are multiplied by under ``scaling``: 0.1 ln(factor) + 1 for "yarn", else 1."""
+    if scaling is not None and scaling.get("kind") == "yarn":
+        return 0.1 * math.log(float(scaling["factor"])) + 1.0
+    return 1.0
+
+
 @register_part("position", "rotary")
 class Rotary(PositionEncoding):
     """params: rotary_dim, theta, scaling (mapping or None), pairing ("half"|"interleaved")."""
@@ -63,6 +84,8 @@ class Rotary(PositionEncoding):
             raise ValueError(f"rotary_dim {self.rotary_dim} must be even")
         self.theta = float(p["theta"])
         self.scaling = p.get("scaling")
+        if rotary_length(self.scaling) != 1.0:
+            raise ValueError("rotary: the kernels of this part turn vectors without lengthening them")
         pairing = p.get("pairing", "half")
         if pairing not in ("half", "interleaved"):
             raise ValueError(f"rotary pairing {pairing!r} is not known (half, interleaved)")

@@ -260,6 +260,8 @@ class EmuKernels:
     def add_grouped_rmsnorm(self, x, delta, through, rows, weight, groups, eps, out):
         def norm(v, w):
             v = v.to(self.math)
+            if w is None:
+                return v
             parts = v.reshape(v.shape[0], groups, v.shape[1] // groups)
             return (parts * torch.rsqrt(parts.pow(2).mean(-1, keepdim=True) + eps)).reshape(v.shape) * w.to(self.math)
 
@@ -340,10 +342,10 @@ class EmuKernels:
 
     def latent_prepare(self, proj, n_q, positions, token_row, c_weight, eps, inv_freq, rot_dims, heads, dim, rot_dim, rank, head_dim,
                        q_lat, k_cache, block_table, page_size, write_cache, q_off=None, row_out=None, half_pairs=False,
-                       latent=None):
+                       latent=None, rot_mult=1.0):
         t, m = proj.shape[0], self.math
         ang = positions.to(torch.float32)[:, None] * inv_freq.to(torch.float32)[None, :]
-        cos, sin = ang.cos().to(m), ang.sin().to(m)
+        cos, sin = (ang.cos() * rot_mult).to(m), (ang.sin() * rot_mult).to(m)
 
         def rotate(v):                      # [..., rot_dim] with t leading
             shape = (t,) + (1,) * (v.dim() - 2) + (rot_dims // 2,)
@@ -359,6 +361,8 @@ class EmuKernels:
         ql = q_lat[:, : heads * head_dim].view(t, heads, head_dim)
         ql[:, :, q_off: q_off + rot_dim] = rotate(q[..., dim:]).to(q_lat.dtype)
         ql[:, :, q_off + rot_dim:] = 0
+        if not write_cache and row_out is None:
+            return
         down = (proj[:, n_q: n_q + rank + rot_dim] if latent is None else latent[:, : rank + rot_dim]).to(m)
         c = down[:, :rank]
         c = c * torch.rsqrt(c.pow(2).mean(-1, keepdim=True) + eps) * c_weight.to(m)
@@ -450,7 +454,8 @@ class EmuKernels:
                 state[slot] = seq[-k:].to(state.dtype)
 
     def linear_recurrence(self, mode, q, k, v, state, ctx, out, heads, qk_heads, dk, dv, aux=None, rate=None, decay=None,
-                          a_log=None, dt_bias=None, d_skip=None, q_scale=1.0, rate_per_head=False, bonus=None, rate_scale=1.0):
+                          a_log=None, dt_bias=None, d_skip=None, q_scale=1.0, rate_per_head=False, bonus=None, rate_scale=1.0,
+                          inv_freq=None, rot_dims=0, k_scale=1.0):
         m = self.math
         f = torch.nn.functional
         cu = ctx.cu_q.tolist()
@@ -462,7 +467,16 @@ class EmuKernels:
             kk = k[a:b, : qk_heads * dk].to(m).reshape(n, qk_heads, dk).repeat_interleave(rep, 1)
             vv = v[a:b, : heads * dv].to(m).reshape(n, heads, dv)
             s = state[slot].to(m)                                                            # [heads, dk, dv]
-            if mode == "decay":
+            if mode == "retention":
+                half = rot_dims // 2
+                ang = ctx.positions[a:b].to(torch.float32)[:, None] * inv_freq.to(torch.float32)[None, :half]
+                c, sn = ang.cos().to(m)[:, None], ang.sin().to(m)[:, None]
+                turn = lambda z: torch.cat([z[..., :half] * c - z[..., half: rot_dims] * sn, z[..., half: rot_dims] * c + z[..., :half] * sn,
+                                            z[..., rot_dims:]], -1)
+                qq, kk = turn(qq), turn(kk) * k_scale
+                dec = decay.to(m)[None, :, None].expand(n, heads, dk)
+                u_scale = torch.ones(n, heads, dtype=m, device=q.device)
+            elif mode == "decay":
                 qq, kk, vv = f.silu(qq), f.silu(kk), f.silu(vv)
                 dec = decay.to(m)[None, :, None].expand(n, heads, dk)
                 u_scale = torch.ones(n, heads, dtype=m, device=q.device)
@@ -538,15 +552,17 @@ class EmuKernels:
 
     def routed_experts(self, h, logits, w_gate_up, w_down, top, out, score="sigmoid", renormalise=False, scale_input=True,
                        activation="clamped_swish", limit=0.0, alpha=1.702, outputs=None, choice_bias=None, renormalise_eps=0.0,
-                       shared=None, shared_gated=False, weight_scale=1.0):
+                       shared=None, shared_gated=False, weight_scale=1.0, groups=1, keep_groups=1):
         m = self.math
         n_out = logits.shape[1] if outputs is None else outputs
         z = logits[:, :n_out].to(torch.float32)
         scores = torch.sigmoid(z) if score == "sigmoid" else torch.softmax(z, -1)
-        if choice_bias is not None:
-            idx = torch.topk(scores + choice_bias.to(torch.float32), top, dim=-1).indices
-        else:
-            idx = torch.topk(z, top, dim=-1).indices             # by logit: scores of large logits round to ties
+        pick = scores + choice_bias.to(torch.float32) if choice_bias is not None else z      # by logit: scores of large logits round to ties
+        if groups > 1:
+            best = pick.reshape(pick.shape[0], groups, -1).amax(-1)
+            closed = torch.ones_like(best, dtype=torch.bool).scatter(1, torch.topk(best, keep_groups, dim=-1).indices, False)
+            pick = pick.masked_fill(closed.repeat_interleave(n_out // groups, 1), float("-inf"))
+        idx = torch.topk(pick, top, dim=-1).indices
         wts = torch.gather(scores, 1, idx)
         if renormalise:
             wts = wts / (wts.sum(-1, keepdim=True) + renormalise_eps)
