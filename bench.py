@@ -11,7 +11,7 @@ of three: the way the reference's own benchmark times its generate()); ``prefill
 compares the decode step with the bytes it has to read (every weight once, and the cache of the live requests).
 The weights (2.47 GB) are larger than the L2 cache, so no flush is needed between steps.
 
-``--design rogisun`` (or ``bapavik``, ``lilunex``, ``gebilorn``, ``vivepel``) is another measurement altogether and leaves the line above as it
+``--design rogisun`` (or ``bapavik``, ``lilunex``, ``gebilorn``, ``vivepel``, ``filezen``) is another measurement altogether and leaves the line above as it
 is: prefill and decode throughput of the Rogisun decoder (three layers, one of each mixer, routed experts) at layer sizes of real models,
 beside a Llama decoder of equal width, depth and active feed-forward size, each with the device time of every kernel
 of one prompt step and one decoding step; it prints its own JSON line (see design_bench).
@@ -421,7 +421,26 @@ def vivepel_at(width: int, vocab: int = 32000):
                              "max_position": CONTEXT})
 
 
-DESIGNS = {"rogisun": rogisun_at, "bapavik": bapavik_at, "lilunex": lilunex_at, "gebilorn": gebilorn_at, "vivepel": vivepel_at}
+def filezen_at(width: int, vocab: int = 32000):
+    """A Filezen configuration with layers of a real model's sizes: latent attention (cached rows of 192 + 64, heads of 128 + 64, a
+    window of 1,024 keys, scaled frequencies) with experts in eight groups and a shared expert; retention (heads of 128 x 128) with a
+    dense feed-forward; latent attention on the first layer's rows with experts."""
+    from serve_b200.config import config_from_dict
+
+    heads, experts, top, ff = DESIGN_SIZES[str(width)]
+    moe = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top, "groups": {"count": 8, "keep": 4}}, "shared": {"ff": ff}}
+    lat = {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 192, "scale": 192 ** -0.5, "mask": {"size": 1024},
+           "rot": {"base": 10000.0, "dims": 64, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    ret = {"heads": heads, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-5.0 - 4.0 * h / heads) for h in range(heads)],
+           "rot": {"base": 10000.0, "dims": 128}}
+    layers = [{"type": "latent_attention", "mixer": lat, "mlp": moe}, {"type": "retention", "mixer": ret, "mlp": {"kind": "dense", "ff": top * ff}},
+              {"type": "latent_attention", "mixer": dict(lat, kv_from=0), "mlp": moe}]
+    return config_from_dict({"architecture": "Filezen", "width": width, "vocab": vocab, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
+                             "residual_mult": 0.5, "layers": layers, "max_position": CONTEXT})
+
+
+DESIGNS = {"rogisun": rogisun_at, "bapavik": bapavik_at, "lilunex": lilunex_at, "gebilorn": gebilorn_at, "vivepel": vivepel_at,
+           "filezen": filezen_at}
 
 
 def kernel_times(eng, entries, end):
@@ -468,7 +487,7 @@ def prefill_many(eng, vocab, requests, each, reps=5, seed=11):
 
 def design_bench(args):
     """Prefill (one prompt of 2,048 tokens) and decode (batch 8 after 2,048-token prompts, from CUDA graphs) of the named design
-    (Rogisun, Bapavik, Lilunex, Gebilorn or Vivepel) and of the Llama decoder of equal size, at each width asked for, bfloat16, random weights; CUDA events on the stream, the
+    (Rogisun, Bapavik, Lilunex, Gebilorn, Vivepel or Filezen) and of the Llama decoder of equal size, at each width asked for, bfloat16, random weights; CUDA events on the stream, the
     weights alone exceed the L2 cache. Prints one JSON line: per width and design the two rates, the rate of a step of 8 prompts
     of 256 tokens (the same tokens side by side: what a recurrence walks in turn for one prompt it walks at once for eight),
     and the kernels of one prompt step and one (eager) decoding step with their device times."""

@@ -335,7 +335,7 @@ class EmuKernels:
         if temp_coef:
             temp = 1.0 + temp_coef * torch.log((torch.div(positions.long() + 1, temp_every, rounding_mode="floor") + 1).to(torch.float32))
             q = q * temp.to(m)[:, None]
-        x[:, :heads] = q.view(t, heads, d).to(proj.dtype)
+        x[:, :heads] = q.view(t, heads, d).to(proj.dtype).clone()      # (q may be a view of x)
         if write_cache:
             self._write_pages(k_cache, k.view(t, kv_heads, d), positions, token_row, block_table, page_size)
             self._write_pages(v_cache, x[:, heads + kv_heads:], positions, token_row, block_table, page_size)
