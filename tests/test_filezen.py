@@ -265,7 +265,7 @@ def test_latent_attention_alone(backend, cuts, which):
 
 
 @pytest.mark.parametrize("backend", BACKENDS)
-@pytest.mark.parametrize("cuts", CUTS, ids=["whole", "portions", "tokens"])
+@pytest.mark.parametrize("cuts", CUTS + [[33, 2, 130, 1, 64, 40]], ids=["whole", "portions", "tokens", "long-portions"])
 @pytest.mark.parametrize("which", range(len(RETS)))
 def test_retention_alone(backend, cuts, which):
     """Also: a head that never forgets, one that sees the current token only; a state taller than wide and wider than tall;
@@ -565,6 +565,69 @@ def test_states_of_a_slot_are_the_next_requests(backend):
             mgr.close(rid)
     want = _plain_mixer("retention", x.double(), F64(w), m, 1e-2).float()
     torch.testing.assert_close(outs[1], want, atol=2 * _tol(backend, want), rtol=0)
+
+
+# ---- the chunked form of the recurrence -----------------------------------------------------------------------------
+@pytest.mark.gpu
+@pytest.mark.parametrize("listed", [True, False], ids=["rows-by-length", "rows-in-order"])
+@pytest.mark.parametrize("lens,heads,dk,dv,rot,decay", [
+    ([100, 1, 33, 64, 65, 2, 300, 32], 3, 32, 32, 32, [0.97, 0.9, 0.999]), ([40], 2, 64, 96, 16, [1.0, 0.0]), ([200, 70], 2, 20, 24, 8, [0.5, 0.99]),
+    ([90, 33], 1, 128, 72, 64, [0.98]), ([500, 1, 1], 4, 16, 16, 0, [0.9, 0.99, 0.999, 1.0]), ([129, 32], 2, 8, 100, 8, [0.8, 0.2]),
+    ([128, 257], 2, 128, 128, 128, [0.99, 0.9995])])
+def test_recurrence_chunk_by_chunk_in_one_batch(lens, heads, dk, dv, rot, decay, listed):
+    """A ragged step on states that hold something already, positions that do not start at zero, slots in another order than
+    the rows: read-outs and last states equal the recurrence in float64 on the same bfloat16 operands, for lengths below, at and
+    just above the threshold, one and several chunks, and chunks that are filled partly. What enters the recurrence is not rounded
+    again, so the agreement is that of 32-bit sums."""
+    from types import SimpleNamespace
+
+    from serve_b200.engine.step import BatchShape
+    from serve_b200.kernels import load_kernels
+
+    k, dev = load_kernels("cuda:0"), "cuda:0"
+    g = torch.Generator().manual_seed(sum(lens))
+    t, rows = sum(lens), len(lens)
+    cu = [0]
+    for n in lens:
+        cu.append(cu[-1] + n)
+    starts = [11 * i + 3 for i in range(rows)]
+    proj = torch.randn(t, 2 * heads * dk + 2 * heads * dv, generator=g).bfloat16()
+    state0 = torch.randn(rows, heads, dk, dv, generator=g)
+    inv = torch.tensor([100.0 ** (-2.0 * i / max(rot, 1)) for i in range(max(rot // 2, 1))])
+    order = sorted(range(rows), key=lambda i: -lens[i])
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    shape = BatchShape(rows, t, max(lens), min(lens), 4096, False, rows_by_q=i32(order) if listed else None,
+                       neg_q_sorted=tuple(-lens[i] for i in order) if listed else None)
+    slots = list(range(rows))[::-1]
+    ctx = SimpleNamespace(shape=shape, positions=i32([s + j for n, s in zip(lens, starts) for j in range(n)]),
+                          token_row=i32([i for i, n in enumerate(lens) for _ in range(n)]), cu_q=i32(cu), slots=i32(slots), memo={})
+    q, kk, v = proj[:, : heads * dk], proj[:, heads * dk: 2 * heads * dk], proj[:, 2 * heads * dk: 2 * heads * dk + heads * dv]
+    on = proj.to(dev)
+    part = lambda a, n: on[:, a: a + n]
+    state = state0.to(dev)
+    out = torch.full((t, heads * dv), float("nan"), device=dev)
+    before = k.launches
+    k.linear_recurrence("retention", part(0, heads * dk), part(heads * dk, heads * dk), part(2 * heads * dk, heads * dv), state, ctx, out, heads, heads,
+                        dk, dv, decay=torch.tensor(decay, device=dev), inv_freq=inv.to(dev), rot_dims=rot, k_scale=dk ** -0.5)
+    assert k.launches - before == 3 + (1 if rot else 0) + (2 if min(lens) <= k.CHUNKED_FROM else 0)
+    for r, n in enumerate(lens):
+        sl = slice(cu[r], cu[r + 1])
+        ang = (torch.arange(n) + starts[r]).float()[:, None] * inv[None, : rot // 2]          # (angles are 32-bit)
+        c, sn = ang.double().cos()[:, None], ang.double().sin()[:, None]
+
+        def turn(z):
+            z = z[sl].double().view(n, heads, dk)
+            a, b = z[..., : rot // 2], z[..., rot // 2: rot]
+            return torch.cat([a * c - b * sn, b * c + a * sn, z[..., rot:]], -1)
+
+        qq, ke, ve = turn(q), turn(kk) * dk ** -0.5, v[sl].double().view(n, heads, dv)
+        S = state0[slots[r]].double()
+        want = torch.zeros(n, heads, dv).double()
+        for i in range(n):
+            S = torch.tensor(decay).double()[:, None, None] * S + ke[i][:, :, None] * ve[i][:, None, :]
+            want[i] = torch.einsum("hkv,hk->hv", S, qq[i])
+        torch.testing.assert_close(out[sl].cpu().double(), want.view(n, heads * dv), atol=3e-5 * float(want.abs().max()), rtol=0)
+        torch.testing.assert_close(state[slots[r]].cpu().double(), S, atol=2e-5 * float(S.abs().max()), rtol=0)
 
 
 # ---- the sizes of a real layer, and the programs a user starts ----------------------------------------------------
